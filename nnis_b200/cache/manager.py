@@ -5,12 +5,13 @@ once (a tuple of requests: a layer whose mixer is made of two, say; its view is 
 their views, in the same order):
 
 * ``KVRequest`` - keys and values of every position (``window == 0``) or of the
-  last ``window`` positions.  Entries with the same (kv_heads, head_dim, window)
-  form a *group* with storage and a page pool of its own:
+  last ``window`` positions.  Entries with the same (kv_heads, head_dim, window, kept
+  first tokens) form a *group* with storage and a page pool of its own:
   ``k, v: [entries, pages, kv_heads, page_size, head_dim]``.  A page id is
   valid for every entry of its group, so one page table per group and sequence
   serves all its layers.  A windowed group gives pages back as soon as they fall
-  wholly out of the window.
+  wholly out of the window.  With ``keep_first`` the pages that hold a sequence's first
+  ``keep_first`` positions stay all the same (a window that keeps the first tokens).
   With ``values=False`` the group keeps one tensor only (``v`` is None): rows that
   serve as keys and carry the values inside them, as latent attention's do.
   ``value_dim`` gives the values a size of their own (0: the keys' size).
@@ -44,6 +45,7 @@ class KVRequest:
     window: int = 0
     values: bool = True  # False: no storage for values (the key rows carry them)
     value_dim: int = 0  # size of a value head; 0: head_dim
+    keep_first: int = 0  # first positions of a sequence that a windowed group keeps
 
 
 @dataclass(frozen=True)
@@ -71,6 +73,7 @@ class KVView:
     v: Optional[torch.Tensor]  # [pages, kv_heads, page_size, value_dim]; None for a group without values
     page_size: int
     window: int
+    keep_first: int = 0
     ahead: int = 0  # elements from k (and v) to those of the group's layer that runs next; 0: none
 
 
@@ -81,9 +84,10 @@ class StateView:
 
 
 class _KVGroup:
-    def __init__(self, key: Tuple[int, int, int, bool, int], entries: List[int], pages: int,
+    def __init__(self, key: Tuple[int, int, int, bool, int, int], entries: List[int], pages: int,
                  dtype: torch.dtype, device: torch.device):
-        self.kv_heads, self.head_dim, self.window, self.values, self.value_dim = key
+        self.kv_heads, self.head_dim, self.window, self.values, self.value_dim, self.keep_first = key
+        self.kept_pages = -(-self.keep_first // PAGE_SIZE)  # these never go back while the sequence lives
         self.entries = entries
         self.pool = FreeList(pages, "page")
         shape = (len(entries), pages, self.kv_heads, PAGE_SIZE, self.head_dim)
@@ -93,7 +97,7 @@ class _KVGroup:
         self.tables: Dict[int, List[int]] = {}
 
     def first_needed_page(self, length: int) -> int:
-        """Pages before this one hold no key that a later position may read."""
+        """Pages before this one (but for the kept first ones) hold no key that a later position may read."""
         if self.window <= 0:
             return 0
         return max(0, length - self.window + 1) // PAGE_SIZE if length > 0 else 0
@@ -120,7 +124,7 @@ class CacheManager:
         self.owners: List[int] = [0] * max_slots  # how many sequences have held each slot
         self.groups: List[_KVGroup] = []
         self._views: List[Optional[Union[KVView, StateView]]] = []
-        by_key: Dict[Tuple[int, int, int, bool, int], List[int]] = {}
+        by_key: Dict[Tuple[int, int, int, bool, int, int], List[int]] = {}
         # an entry that asks for several things: each is served like an entry's own request, and
         # the entry's view is the tuple of what they get
         spans: List[Optional[Tuple[int, int]]] = []
@@ -136,7 +140,8 @@ class CacheManager:
         for i, r in enumerate(requests):
             if isinstance(r, KVRequest):
                 by_key.setdefault((r.kv_heads, r.head_dim, r.window, bool(r.values),
-                                   (r.value_dim or r.head_dim) if r.values else 0), []).append(i)
+                                   (r.value_dim or r.head_dim) if r.values else 0,
+                                   r.keep_first if r.window > 0 else 0), []).append(i)
         group_of: Dict[int, Tuple[int, int]] = {}
         for key, entries in by_key.items():
             g = _KVGroup(key, entries, self.pages_total, dtype, self.device)
@@ -150,7 +155,7 @@ class CacheManager:
                 g = self.groups[gi]
                 nxt = (j + 1) % len(g.entries)  # (after the last layer: the first, in the next step)
                 self._views.append(KVView(gi, g.k[j], g.v[j] if g.values else None, PAGE_SIZE, g.window,
-                                          (nxt - j) * g.k[0].numel()))
+                                          g.keep_first, (nxt - j) * g.k[0].numel()))
             elif isinstance(r, StateRequest):
                 made = [torch.zeros((max_slots, *shape), dtype=dtype, device=self.device)
                         for shape, dtype in ((r.shape, r.dtype), *r.extra)]
@@ -239,7 +244,7 @@ class CacheManager:
             for g in self.groups:
                 if g.window > 0:
                     table = g.tables[slot]
-                    for i in range(min(g.first_needed_page(n), len(table))):
+                    for i in range(g.kept_pages, min(g.first_needed_page(n), len(table))):
                         if table[i] >= 0:
                             g.pool.give(table[i])
                             table[i] = -1

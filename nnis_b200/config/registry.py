@@ -18,6 +18,7 @@ from .llama import ConfigError, LlamaConfig
 from .nafezen import NafezenConfig
 from .sedopel import SedopelConfig
 from .selovik import SelovikConfig
+from .setenex import SetenexConfig
 from .tazadra import TazadraConfig
 from .spec import ModelSpec
 
@@ -87,3 +88,4 @@ register_architecture(NafezenConfig.architecture, NafezenConfig)
 register_architecture(TazadraConfig.architecture, TazadraConfig)
 register_architecture(SedopelConfig.architecture, SedopelConfig)
 register_architecture(SelovikConfig.architecture, SelovikConfig)
+register_architecture(SetenexConfig.architecture, SetenexConfig)

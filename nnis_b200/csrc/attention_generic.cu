@@ -142,7 +142,7 @@ static int launch_attention(const void* q, int q_stride, const void* k_cache, co
     if (n_splits > 1) {
         size_t rows = (size_t)n_tokens * nq;
         attn_merge_kernel<T><<<(unsigned)rows, 128, 0, stream>>>(partial, (T*)out, rows,
-                                                                             d, n_splits);
+                                                                             d, n_splits, nullptr);
     }
     NNIS_RETURN_LAUNCH();
 }
@@ -154,7 +154,7 @@ extern "C" int nnis_attention_merge_bf16(const float* partial, void* out, long l
                                          int n_splits, cudaStream_t stream) {
     if (n_splits > 64) return NNIS_ERR_UNSUPPORTED;
     nnis::attn_merge_kernel<nnis::bf16><<<(unsigned)n_rows, 128, 0, stream>>>(
-        partial, (nnis::bf16*)out, (size_t)n_rows, d, n_splits);
+        partial, (nnis::bf16*)out, (size_t)n_rows, d, n_splits, nullptr);
     NNIS_RETURN_LAUNCH();
 }
 

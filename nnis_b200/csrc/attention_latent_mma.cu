@@ -13,6 +13,10 @@
 // softmax between the products is float32 in registers.  Rows in shared memory are padded
 // to a multiple of 64 values (zeros) so that the XOR swizzle stays inside a row.
 //
+// With `window` a query at position p sees keys above p - window only, and the walk begins at
+// the page of the first key that the tile's first row sees.  `gate` (float32, one per stacked
+// row) multiplies the row's output.
+//
 // The key range may be cut into slices (blockIdx.z), for steps with few rows and long
 // contexts: a slice leaves [max, sum, unnormalised output] per row and the merge kernel
 // adds the slices up in order.
@@ -40,7 +44,7 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
                   const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                   const int* __restrict__ page_table, int table_cols, bf16* __restrict__ out,
                   float* __restrict__ partial, int heads, int dk, int dv, int dkp, int tiles_per_token,
-                  float scale, int n_splits) {
+                  float scale, int n_splits, int window, const float* __restrict__ gate) {
     constexpr int KH = NT == 16 ? 64 : 32, KB = KH / 8, RUN = NT * 8;
     constexpr int TILE = SPLIT_ROWS ? 2 * kLatRows : kLatRows;  // rows of the CTA
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -79,10 +83,11 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
         return;  // (a padding row: the merge and the projections after it read nothing of it)
     }
     const int hi = start + (r0 + rows - 1) / heads + 1;  // keys below this position may be seen
-    const int all_pages = (hi - 1) / kLatPage + 1;
-    const int per = (all_pages + n_splits - 1) / n_splits;
-    const int first_page = split * per;
-    const int n_pages = max(0, min(all_pages, first_page + per) - first_page);
+    const int end_page = (hi - 1) / kLatPage + 1;
+    const int seen_page = window > 0 ? max(0, start + r0 / heads - window + 1) / kLatPage : 0;
+    const int per = (end_page - seen_page + n_splits - 1) / n_splits;
+    const int first_page = seen_page + split * per;
+    const int n_pages = max(0, min(end_page, first_page + per) - first_page);
     const int* table = page_table + (size_t)seq * table_cols;
     const size_t tile_elems = (size_t)kLatPage * dkp;
 
@@ -120,6 +125,9 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
 #pragma unroll
     for (int h = 0; h < 2; ++h) pos_r[h] = start + (r0 + g_row + warp * 16 + r_lo + h * 8) / heads;
     const int warp_last_pos = start + (r0 + g_row + warp * 16 + 15) / heads;
+    // (the first key that any of the warp's rows sees; far below zero without a window)
+    const int reach = window > 0 ? window : 0x3fffffff;
+    const int warp_first_key = start + (r0 + g_row + warp * 16) / heads - reach + 1;
     float o[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; ++j)
@@ -135,12 +143,14 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
         load_page(it + STAGES - 1);
         const bf16* kt = k_s + (size_t)(it % STAGES) * tile_elems;
         const int t0 = (first_page + it) * kLatPage;
-        if (t0 > warp_last_pos || dv_here <= 0) continue;  // none of this warp's rows sees the page
+        // none of this warp's rows sees the page
+        if (t0 > warp_last_pos || t0 + kLatPage <= warp_first_key || dv_here <= 0) continue;
 
 #pragma unroll
         for (int half = 0; half < kLatPage / KH; ++half) {
             const int tk = t0 + half * KH;  // first key of this softmax step
             if (tk > warp_last_pos) break;
+            if (tk + KH <= warp_first_key) continue;
             float s[KB][4];
 #pragma unroll
             for (int j = 0; j < KB; ++j)
@@ -165,7 +175,7 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     int key = tk + j * 8 + c_lo + (e & 1);
-                    float v = key <= pos_r[e >> 1] ? s[j][e] * sc : -INFINITY;
+                    float v = key <= pos_r[e >> 1] && key > pos_r[e >> 1] - reach ? s[j][e] * sc : -INFINITY;
                     s[j][e] = v;
                     mx[e >> 1] = fmaxf(mx[e >> 1], v);
                 }
@@ -217,8 +227,12 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
     }
     const int ra = g_row + warp * 16 + r_lo, rb = ra + 8;
     if (n_splits == 1) {
-        const float inv_a = l_run[0] > 0.f ? 1.0f / l_run[0] : 0.f;
-        const float inv_b = l_run[1] > 0.f ? 1.0f / l_run[1] : 0.f;
+        float inv_a = l_run[0] > 0.f ? 1.0f / l_run[0] : 0.f;
+        float inv_b = l_run[1] > 0.f ? 1.0f / l_run[1] : 0.f;
+        if (gate) {
+            if (ra < rows) inv_a *= gate[row_base + ra];
+            if (rb < rows) inv_b *= gate[row_base + rb];
+        }
 #pragma unroll
         for (int jn = 0; jn < NT; ++jn) {
             int col = jn * 8 + c_lo;
@@ -286,14 +300,16 @@ NNIS_API int nnis_attention_latent_mma_tile_rows(int dv) { return latent_tile_ro
 // rows per tile, with the per-sequence first packed row, first position and token count; or
 // null, and then every row of the step is one token of a sequence of its own (n_tokens
 // rows, ceil(heads / tile rows) tiles each).
-// `partial`: float32 [n_tokens * heads * n_splits * (dv + 2)] when n_splits > 1.
+// `partial`: float32 [n_tokens * heads * n_splits * (dv + 2)] when n_splits > 1.  `gate`: float32
+// [n_tokens, heads] or null.
 NNIS_API int nnis_attention_latent_mma(const void* q, const void* cache, const int* tiles, int n_tiles,
                                        const int* seq_first_row, const int* seq_start,
                                        const int* seq_count, const int* token_pos, const int* token_seq,
                                        const int* page_table, int table_cols, void* out, float* partial,
                                        int n_tokens, int heads, int dk, int dv, int page_size,
-                                       float scale, int n_splits, cudaStream_t stream) {
-    if (n_tokens <= 0 || heads <= 0 || table_cols <= 0 || n_splits <= 0 || !q || !cache || !out ||
+                                       float scale, int n_splits, int window, const float* gate,
+                                       cudaStream_t stream) {
+    if (n_tokens <= 0 || heads <= 0 || table_cols <= 0 || n_splits <= 0 || window < 0 || !q || !cache || !out ||
         !page_table)
         return NNIS_ERR_ARGUMENT;
     if (!nnis_attention_latent_mma_takes(dk, dv, page_size)) return NNIS_ERR_UNSUPPORTED;
@@ -311,7 +327,8 @@ NNIS_API int nnis_attention_latent_mma(const void* q, const void* cache, const i
     const int stages = latent_mma_smem(dk, dv, 3) <= 200 * 1024 ? 3 : 2;
     const size_t smem = latent_mma_smem(dk, dv, stages);
     using Kernel = void (*)(const bf16*, const bf16*, const int*, const int*, const int*, const int*, const int*,
-                            const int*, const int*, int, bf16*, float*, int, int, int, int, int, float, int);
+                            const int*, const int*, int, bf16*, float*, int, int, int, int, int, float, int, int,
+                            const float*);
     Kernel kernel;
     if (run == 128) kernel = stages == 3 ? latent_mma_kernel<3, 16, true> : latent_mma_kernel<2, 16, true>;
     else if (split_rows) kernel = stages == 3 ? latent_mma_kernel<3, 32, true> : latent_mma_kernel<2, 32, true>;
@@ -323,12 +340,12 @@ NNIS_API int nnis_attention_latent_mma(const void* q, const void* cache, const i
     cudaError_t e = launch_dependent(kernel, grid, 256, smem, stream, (const bf16*)q, (const bf16*)cache, tiles,
                                      seq_first_row, seq_start, seq_count, token_pos, token_seq, page_table,
                                      table_cols, (bf16*)out, partial, heads, dk, dv, dkp, tiles_per_token, scale,
-                                     n_splits);
+                                     n_splits, window, gate);
     if (e != cudaSuccess) return (int)e;
     if (n_splits > 1) {
         size_t rows = (size_t)n_tokens * heads;
         e = launch_dependent(attn_merge_kernel<bf16>, (unsigned)rows, 128, 0, stream, (const float*)partial,
-                             (bf16*)out, rows, dv, n_splits);
+                             (bf16*)out, rows, dv, n_splits, gate);
     }
     return e == cudaSuccess ? NNIS_OK : (int)e;
 }

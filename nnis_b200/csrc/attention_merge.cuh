@@ -1,6 +1,7 @@
 // The merge of split attention: kernels that cut a query's key range into slices
 // leave, per (token, head, slice), a record [running max, running sum, unnormalised
-// output of d values]; this kernel adds the slices up in ascending order.
+// output of d values]; this kernel adds the slices up in ascending order.  With `row_gate`
+// (float32, one per row) the row's output is multiplied by it.
 #pragma once
 
 #include <float.h>
@@ -16,7 +17,7 @@ namespace nnis {
 template <typename T>
 __global__ void __launch_bounds__(128)
 attn_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, size_t n_rows, int d,
-                  int n_splits) {
+                  int n_splits, const float* __restrict__ row_gate) {
     __shared__ float share[64];
     pdl_wait();  // (a no-op unless launched as a programmatic dependent)
     pdl_launch_dependents();
@@ -41,7 +42,8 @@ attn_merge_kernel(const float* __restrict__ partial, T* __restrict__ out, size_t
             l += ls[k] * ms[k];
         }
         l = warp_sum(l);
-        const float inv = l > 0.f ? 1.0f / l : 0.f;
+        float inv = l > 0.f ? 1.0f / l : 0.f;
+        if (row_gate) inv *= row_gate[row];
         share[lane] = ms[0] * inv;
         share[lane + 32] = ms[1] * inv;
     }

@@ -1,6 +1,7 @@
-// Attention with a soft cap on its scores, a sink in the softmax's denominator, a chunked
-// or windowed causal mask, key and value heads of different sizes and a gate per head, over
-// the paged cache; and the row-wise step in front of it.
+// Attention with a soft cap on its scores, a learned bias per distance, a sink in the softmax's
+// denominator, a chunked or windowed causal mask that may keep the first tokens, key and value
+// heads of different sizes and a gate per head, over the paged cache; and the row-wise step in
+// front of it.
 //
 //   qkv_prep        from the projection's float32 rows [q (H dk) | k (G dk) | v (G dv) | gate (H)]:
 //                   RMS norm of q and of k over the WHOLE projection (all heads at once, one
@@ -10,8 +11,9 @@
 //                   is optional (no norm weights, rot 0, no k/v in the rows, no gate).
 //   qkv_prep_heads  the same step with everything per head: rotation of either pairing (neighbours, or
 //                   value i with value i + rot / 2), then optionally an RMS norm of every q and k head
-//                   by itself (no weight, after the rotation), optionally a number per query head that
-//                   multiplies its q (a temperature of the scores), and `gate_cols` gate logits a token
+//                   by itself (no weight, after the rotation) or an RMS norm with a weight per value of
+//                   a head, shared by the heads (wq, wk, before the rotation), optionally a number per query
+//                   head that multiplies its q (a temperature of the scores), and `gate_cols` gate logits a token
 //                   (one per head, or one per output value).  A head may hold `maps` vectors of equal
 //                   size side by side (the queries and keys of several attention maps over one set of
 //                   values); each is turned by itself over its own first `rot` values.  `magnitude`
@@ -20,7 +22,9 @@
 //                   an online softmax in float32: score = cap * tanh(scale * q.k / cap) (cap 0: none);
 //                   a query at position p sees keys j <= p with j >= p - window + 1 (window > 0) and
 //                   floor(j / chunk) == floor(p / chunk) (chunk > 0, chunks counted from position 0 of
-//                   the sequence); the denominator also holds exp(sink[head]), which has no key and
+//                   the sequence), and the keys j < keep whatever window and chunk say; with `bias`
+//                   (a table of `bias_len` distances per query head) a score gains, after scale and cap,
+//                   bias[head][min(p - j, bias_len - 1)]; the denominator also holds exp(sink[head]), which has no key and
 //                   no value; the output is multiplied by gate[token, head] (or, with `gate_elems` = dv, value by value
 //                   by gate[token, head, :]).  The key range may be
 //                   cut into slices whose partial records a second kernel merges in order (the sink
@@ -116,7 +120,8 @@ qkv_prep_kernel(const float* __restrict__ a, const float* __restrict__ wq, const
 // A warp per head of q and of k.  pairing 0: values (2i, 2i + 1) turn together; 1: values (i, i + rot / 2).
 template <typename T>
 __global__ void __launch_bounds__(256)
-qkv_prep_heads_kernel(const float* __restrict__ a, const float* __restrict__ q_scale,
+qkv_prep_heads_kernel(const float* __restrict__ a, const float* __restrict__ wq, const float* __restrict__ wk,
+                      const float* __restrict__ q_scale,
                       const float* __restrict__ freq, const int* __restrict__ token_pos,
                       const int* __restrict__ token_seq, const int* __restrict__ page_table, int table_cols,
                       T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
@@ -144,6 +149,13 @@ qkv_prep_heads_kernel(const float* __restrict__ a, const float* __restrict__ q_s
         const bool is_q = hh < H;
         const int h = is_q ? hh : hh - H;
         const float* src = row + (is_q ? 0 : nq) + (size_t)h * dk;
+        const float* wn = is_q ? wq : wk;
+        float before = 1.0f;  // one over the head's root mean square, with a norm before the rotation
+        if (wn) {
+            float ss = 0.f;
+            for (int i = lane; i < dk; i += 32) ss = fmaf(src[i], src[i], ss);
+            before = 1.0f / sqrtf(warp_sum(ss) / (float)dk + eps);
+        }
         // a lane takes a pair: one cosine and one sine serve both of its values, and every map's pair
         // of the same place turns by the same angle
         for (int f = lane; f < half; f += 32) {
@@ -153,13 +165,18 @@ qkv_prep_heads_kernel(const float* __restrict__ a, const float* __restrict__ q_s
             c *= magnitude;
             for (int base = 0; base < dk; base += sub) {
                 const int i0 = base + (pairing ? f : 2 * f), i1 = pairing ? i0 + half : i0 + 1;
-                const float x0 = src[i0], x1 = src[i1];
+                float x0 = src[i0], x1 = src[i1];
+                if (wn) {
+                    x0 = (x0 * before) * wn[i0];
+                    x1 = (x1 * before) * wn[i1];
+                }
                 buf[i0] = x0 * c - x1 * s;
                 buf[i1] = x1 * c + x0 * s;
             }
         }
         for (int base = 0; base < dk; base += sub)  // (beyond the rotated values of every map)
-            for (int j = rot + lane; j < sub; j += 32) buf[base + j] = src[base + j];
+            for (int j = rot + lane; j < sub; j += 32)
+                buf[base + j] = wn ? (src[base + j] * before) * wn[base + j] : src[base + j];
         float inv = 1.0f;
         if (norm_heads) {
             __syncwarp();
@@ -194,7 +211,8 @@ attn_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
                  const int* __restrict__ page_table, int table_cols, const float* __restrict__ sink,
                  const float* __restrict__ gate, T* __restrict__ out, float* __restrict__ partial,
                  int n_tokens, int nq, int nkv, int dk, int dv, int page_size, int window, int chunk,
-                 float scale, float cap, int n_splits, int gate_elems) {
+                 float scale, float cap, int n_splits, int gate_elems, int keep,
+                 const float* __restrict__ bias, int bias_len) {
     extern __shared__ float q_smem[];
     pdl_wait();
     pdl_launch_dependents();
@@ -218,11 +236,12 @@ attn_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
         __syncwarp();
         int lo = window > 0 ? max(0, pos - window + 1) : 0;
         if (chunk > 0) lo = max(lo, (pos / chunk) * chunk);
-        const int hi = pos + 1;
-        int per = (hi - lo + n_splits - 1) / n_splits;
+        // the visible keys in order: the kept first ones below lo, then lo .. pos
+        const int kept = min(keep, lo), n_keys = kept + pos + 1 - lo, skip = lo - kept;
+        int per = (n_keys + n_splits - 1) / n_splits;
         per = (per + 31) & ~31;
-        const int start = lo + split * per;
-        const int end = min(hi, start + per);
+        const int start = split * per;
+        const int end = min(n_keys, start + per);
         if (sink && split == 0) {  // the sink: a score without a key and without a value
             m = sink[hq];
             l = 1.f;
@@ -230,8 +249,8 @@ attn_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
         const int* table = page_table + (size_t)token_seq[n] * table_cols;
         const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
         for (int c = start; c < end; c += 32) {
-            const int t = c + lane;
-            const bool valid = t < end;
+            const bool valid = c + lane < end;
+            const int t = c + lane < kept ? c + lane : c + lane + skip;
             int row_index = 0;
             float s = -FLT_MAX;
             if (valid) {
@@ -251,6 +270,7 @@ attn_sink_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
                 for (int i = d4; i < dk; ++i) dot = fmaf(qs[i], to_float(krow[i]), dot);
                 s = dot * scale;
                 if (cap > 0.f) s = cap * tanhf(s * inv_cap);
+                if (bias) s += bias[(size_t)hq * bias_len + min(pos - t, bias_len - 1)];
             }
             const float m_new = fmaxf(m, warp_max(s));
             const float p = valid ? expf(s - m_new) : 0.f;
@@ -305,7 +325,8 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
                        const int* __restrict__ page_table, int table_cols, const float* __restrict__ sink,
                        const float* __restrict__ gate, T* __restrict__ out, float* __restrict__ partial,
                        int n_tokens, int nq, int nkv, int dk, int dv, int page_size, int window, int chunk,
-                       float scale, float cap, int n_splits, int gate_elems) {
+                       float scale, float cap, int n_splits, int gate_elems, int keep,
+                       const float* __restrict__ bias, int bias_len) {
     extern __shared__ __align__(16) float q_smem[];
     pdl_wait();
     pdl_launch_dependents();
@@ -333,11 +354,12 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
         __syncwarp();
         int lo = window > 0 ? max(0, pos - window + 1) : 0;
         if (chunk > 0) lo = max(lo, (pos / chunk) * chunk);
-        const int hi = pos + 1;
-        int per = (hi - lo + n_splits - 1) / n_splits;
+        // the visible keys in order: the kept first ones below lo, then lo .. pos
+        const int kept = min(keep, lo), n_keys = kept + pos + 1 - lo, skip = lo - kept;
+        int per = (n_keys + n_splits - 1) / n_splits;
         per = (per + 31) & ~31;
-        const int start = lo + split * per;
-        const int end = min(hi, start + per);
+        const int start = split * per;
+        const int end = min(n_keys, start + per);
         if (sink && split == 0) {
 #pragma unroll
             for (int g = 0; g < G; ++g) {
@@ -349,8 +371,8 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
         const float inv_cap = cap > 0.f ? 1.0f / cap : 0.f;
         const bool by_four = (dk & 3) == 0;
         for (int c = start; c < end; c += 32) {
-            const int t = c + lane;
-            const bool valid = t < end;
+            const bool valid = c + lane < end;
+            const int t = c + lane < kept ? c + lane : c + lane + skip;
             int row_index = 0;
             float s[G];
 #pragma unroll
@@ -385,6 +407,7 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
             for (int g = 0; g < G; ++g) {
                 float sv = s[g] * scale;
                 if (cap > 0.f) sv = cap * tanhf(sv * inv_cap);
+                if (bias && valid) sv += bias[(size_t)(h0 + g) * bias_len + min(pos - t, bias_len - 1)];
                 sv = valid ? sv : -FLT_MAX;
                 const float m_new = fmaxf(m[g], warp_max(sv));
                 p[g] = valid ? expf(sv - m_new) : 0.f;
@@ -394,22 +417,30 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
 #pragma unroll
                 for (int r = 0; r < R; ++r) acc[g][r] *= alpha;
             }
+            // the value rows of several keys are asked for together (beyond the last key: the last row
+            // again, with a weight of zero)
             const int count = min(32, end - c);
-#pragma unroll 2
-            for (int j = 0; j < count; ++j) {
-                const int rj = __shfl_sync(0xffffffffu, row_index, j);
-                const T* vrow = v_cache + (size_t)rj * dv;
-                float vr[R];
+            constexpr int TOGETHER = R >= 4 ? 4 : 8;
+            for (int j0 = 0; j0 < count; j0 += TOGETHER) {
+                float vr[TOGETHER][R];
 #pragma unroll
-                for (int r = 0; r < R; ++r) {
-                    int i = lane + 32 * r;
-                    vr[r] = i < dv ? to_float(vrow[i]) : 0.f;
+                for (int u = 0; u < TOGETHER; ++u) {
+                    const int rj = __shfl_sync(0xffffffffu, row_index, min(j0 + u, count - 1));
+                    const T* vrow = v_cache + (size_t)rj * dv;
+#pragma unroll
+                    for (int r = 0; r < R; ++r) {
+                        int i = lane + 32 * r;
+                        vr[u][r] = i < dv ? to_float(vrow[i]) : 0.f;
+                    }
                 }
 #pragma unroll
-                for (int g = 0; g < G; ++g) {
-                    const float pj = __shfl_sync(0xffffffffu, p[g], j);
+                for (int u = 0; u < TOGETHER; ++u) {
 #pragma unroll
-                    for (int r = 0; r < R; ++r) acc[g][r] = fmaf(pj, vr[r], acc[g][r]);
+                    for (int g = 0; g < G; ++g) {
+                        const float pj = __shfl_sync(0xffffffffu, p[g], j0 + u);
+#pragma unroll
+                        for (int r = 0; r < R; ++r) acc[g][r] = fmaf(pj, vr[u][r], acc[g][r]);
+                    }
                 }
             }
         }
@@ -493,7 +524,7 @@ static int launch_attn_sink(const void* q, const void* k_cache, const void* v_ca
                             const int* token_seq, const int* page_table, int table_cols, const float* sink,
                             const float* gate, void* out, float* partial, int n_tokens, int nq, int nkv, int dk,
                             int dv, int page_size, int window, int chunk, float scale, float cap, int n_splits,
-                            int gate_elems, cudaStream_t stream) {
+                            int gate_elems, int keep, const float* bias, int bias_len, cudaStream_t stream) {
     cudaError_t e;
     const int group = nq / nkv;
     const size_t group_smem = 4 * (size_t)group * dk * sizeof(float);
@@ -504,7 +535,7 @@ static int launch_attn_sink(const void* q, const void* k_cache, const void* v_ca
     e = launch_dependent(attn_sink_group_kernel<T, R, G>, ggrid, 128, group_smem, stream, (const T*)q, \
                          (const T*)k_cache, (const T*)v_cache, token_pos, token_seq, page_table, table_cols, sink, \
                          gate, (T*)out, partial, n_tokens, nq, nkv, dk, dv, page_size, window, chunk, scale, cap, \
-                         n_splits, gate_elems)
+                         n_splits, gate_elems, keep, bias, bias_len)
 #define NNIS_GROUP_R(G) \
     if (dv <= 32) NNIS_GROUP_CASE(1, G); \
     else if (dv <= 64) NNIS_GROUP_CASE(2, G); \
@@ -530,7 +561,7 @@ static int launch_attn_sink(const void* q, const void* k_cache, const void* v_ca
     e = launch_dependent(attn_sink_kernel<T, R>, grid, 128, smem, stream, (const T*)q, (const T*)k_cache, \
                          (const T*)v_cache, token_pos, token_seq, page_table, table_cols, sink, gate, (T*)out, \
                          partial, n_tokens, nq, nkv, dk, dv, page_size, window, chunk, scale, cap, n_splits, \
-                         gate_elems)
+                         gate_elems, keep, bias, bias_len)
     if (dv <= 32) NNIS_SINK_CASE(1);
     else if (dv <= 64) NNIS_SINK_CASE(2);
     else if (dv <= 128) NNIS_SINK_CASE(4);
@@ -578,10 +609,11 @@ NNIS_API int nnis_qkv_prep(const float* a, const float* wq, const float* wk, con
 
 // a: float32 [n, H dk + G dk + G dv + gate_cols]; q_scale: float32 [H] or null; pairing 0: neighbours,
 // 1: halves; norm_heads: every q and k head divided by its own root mean square after the rotation;
+// wq, wk: float32 [dk] or null: a norm of every q (k) head with this weight before the rotation;
 // maps: vectors of dk / maps values side by side in a head, each turned by itself; magnitude: a
 // multiplier of every cosine and sine
-NNIS_API int nnis_qkv_prep_heads(const float* a, const float* q_scale, const float* freq, const int* token_pos,
-                                 const int* token_seq, const int* page_table, int table_cols, void* q_out,
+NNIS_API int nnis_qkv_prep_heads(const float* a, const float* wq, const float* wk, const float* q_scale,
+                                 const float* freq, const int* token_pos, const int* token_seq, const int* page_table, int table_cols, void* q_out,
                                  void* k_cache, void* v_cache, float* gate_out, int n_tokens, int H, int G, int dk,
                                  int dv, int rot, int pairing, int norm_heads, int gate_cols, int page_size,
                                  float eps, int maps, float magnitude, int dtype, cudaStream_t stream) {
@@ -597,13 +629,13 @@ NNIS_API int nnis_qkv_prep_heads(const float* a, const float* q_scale, const flo
     const size_t smem = 8 * (size_t)dk * sizeof(float);
     cudaError_t e;
     if (dtype == NNIS_DTYPE_F32)
-        e = launch_dependent(qkv_prep_heads_kernel<float>, (unsigned)n_tokens, 256, smem, stream, a, q_scale, freq,
-                             token_pos, token_seq, page_table, table_cols, (float*)q_out, (float*)k_cache,
+        e = launch_dependent(qkv_prep_heads_kernel<float>, (unsigned)n_tokens, 256, smem, stream, a, wq, wk, q_scale,
+                             freq, token_pos, token_seq, page_table, table_cols, (float*)q_out, (float*)k_cache,
                              (float*)v_cache, gate_out, H, G, dk, dv, rot, pairing, norm_heads, gate_cols, page_size,
                              eps, maps, magnitude);
     else if (dtype == NNIS_DTYPE_BF16)
-        e = launch_dependent(qkv_prep_heads_kernel<bf16>, (unsigned)n_tokens, 256, smem, stream, a, q_scale, freq,
-                             token_pos, token_seq, page_table, table_cols, (bf16*)q_out, (bf16*)k_cache,
+        e = launch_dependent(qkv_prep_heads_kernel<bf16>, (unsigned)n_tokens, 256, smem, stream, a, wq, wk, q_scale,
+                             freq, token_pos, token_seq, page_table, table_cols, (bf16*)q_out, (bf16*)k_cache,
                              (bf16*)v_cache, gate_out, H, G, dk, dv, rot, pairing, norm_heads, gate_cols, page_size,
                              eps, maps, magnitude);
     else
@@ -613,14 +645,16 @@ NNIS_API int nnis_qkv_prep_heads(const float* a, const float* q_scale, const flo
 
 // q: [n, nq * dk]; caches [pages, nkv, page, dk] and [pages, nkv, page, dv]; sink: float32 [nq] or
 // null; gate: float32 [n, nq] (gate_elems 0 or 1) or [n, nq * dv] (gate_elems = dv) or null; partial:
-// n * nq * n_splits * (dv + 2) floats when n_splits > 1
+// n * nq * n_splits * (dv + 2) floats when n_splits > 1; keep: first keys of a sequence that every
+// later query sees; bias: float32 [nq, bias_len] or null, by distance
 NNIS_API int nnis_attention_sink(const void* q, const void* k_cache, const void* v_cache, const int* token_pos,
                                  const int* token_seq, const int* page_table, int table_cols, const float* sink,
                                  const float* gate, void* out, float* partial, int n_tokens, int nq, int nkv,
                                  int dk, int dv, int page_size, int window, int chunk, float scale, float cap,
-                                 int n_splits, int gate_elems, int dtype, cudaStream_t stream) {
+                                 int n_splits, int gate_elems, int keep, const float* bias, int bias_len,
+                                 int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || nq <= 0 || nkv <= 0 || nq % nkv || page_size <= 0 || table_cols <= 0 || n_splits <= 0 ||
-        window < 0 || chunk < 0 || cap < 0.f)
+        window < 0 || chunk < 0 || cap < 0.f || keep < 0 || (bias && bias_len <= 0))
         return NNIS_ERR_ARGUMENT;
     if (dk <= 0 || dv <= 0 || dk > 1024 || dv > 256) return NNIS_ERR_UNSUPPORTED;
     if (nq > 65535 || n_splits > 64) return NNIS_ERR_UNSUPPORTED;
@@ -629,10 +663,10 @@ NNIS_API int nnis_attention_sink(const void* q, const void* k_cache, const void*
     if (dtype == NNIS_DTYPE_F32)
         return launch_attn_sink<float>(q, k_cache, v_cache, token_pos, token_seq, page_table, table_cols, sink, gate,
                                        out, partial, n_tokens, nq, nkv, dk, dv, page_size, window, chunk, scale,
-                                       cap, n_splits, gate_elems, stream);
+                                       cap, n_splits, gate_elems, keep, bias, bias_len, stream);
     if (dtype == NNIS_DTYPE_BF16)
         return launch_attn_sink<bf16>(q, k_cache, v_cache, token_pos, token_seq, page_table, table_cols, sink, gate,
                                       out, partial, n_tokens, nq, nkv, dk, dv, page_size, window, chunk, scale,
-                                      cap, n_splits, gate_elems, stream);
+                                      cap, n_splits, gate_elems, keep, bias, bias_len, stream);
     return NNIS_ERR_UNSUPPORTED;
 }

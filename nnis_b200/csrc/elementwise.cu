@@ -26,7 +26,7 @@ bool dependent_launches() {
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ tokens,
                              float* __restrict__ hidden, int n_tokens, int width, int vocab,
-                             int* __restrict__ status) {
+                             int* __restrict__ status, float scale) {
     int n = blockIdx.x;
     int token = tokens[n];
     bool bad = token < 0 || token >= vocab;
@@ -36,7 +36,7 @@ __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict_
     }
     const T* row = table + (size_t)token * width;
     float* out = hidden + (size_t)n * width;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) out[i] = bad ? 0.f : to_float(row[i]);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) out[i] = bad ? 0.f : to_float(row[i]) * scale;
 }
 
 // ---------------------------------------------------------------------------
@@ -263,13 +263,15 @@ __global__ void relu2_gate_kernel(const float* __restrict__ u, T* __restrict__ o
 // Rotation of a part of every head by frequencies given as a table: for each
 // token n and head h, the `len` elements at src[n, h * src_head + src_off ...]
 // go to dst[n, h * dst_head + dst_off ...]; the first `dims` of them are turned
-// in pairs (i, i + dims / 2) by the angle pos * freq[i] (float32), the rest pass.
+// in pairs (i, i + dims / 2), or with `neighbours` (2i, 2i + 1), by the angle pos * freq[i]
+// (float32), the rest pass.
 // ---------------------------------------------------------------------------
 template <typename T>
 __global__ void rope_part_kernel(const T* __restrict__ src, long long src_row, int src_head,
                                  int src_off, T* __restrict__ dst, long long dst_row, int dst_head,
                                  int dst_off, const int* __restrict__ token_pos,
-                                 const float* __restrict__ freq, int heads, int len, int dims) {
+                                 const float* __restrict__ freq, int heads, int len, int dims,
+                                 int neighbours) {
     pdl_wait();
     pdl_launch_dependents();
     int n = blockIdx.x;
@@ -281,11 +283,12 @@ __global__ void rope_part_kernel(const T* __restrict__ src, long long src_row, i
         const T* s = src + (size_t)n * src_row + (size_t)h * src_head + src_off;
         T* d = dst + (size_t)n * dst_row + (size_t)h * dst_head + dst_off;
         if (j < half) {
-            float a = to_float(s[j]), b = to_float(s[j + half]);
+            const int i0 = neighbours ? 2 * j : j, i1 = neighbours ? 2 * j + 1 : j + half;
+            float a = to_float(s[i0]), b = to_float(s[i1]);
             float ang = (float)(pos < 0 ? 0 : pos) * freq[j];
             float c = cosf(ang), sn = sinf(ang);
-            d[j] = from_float<T>(a * c - b * sn);
-            d[j + half] = from_float<T>(b * c + a * sn);
+            d[i0] = from_float<T>(a * c - b * sn);
+            d[i1] = from_float<T>(b * c + a * sn);
         } else {
             d[j + half] = s[j + half];
         }
@@ -310,15 +313,15 @@ NNIS_API int nnis_stream_synchronize(cudaStream_t stream) {
 }
 
 NNIS_API int nnis_embed(const void* table, int dtype, const int* tokens, float* hidden,
-                        int n_tokens, int width, int vocab, int* status, cudaStream_t stream) {
+                        int n_tokens, int width, int vocab, int* status, float scale, cudaStream_t stream) {
     if (n_tokens <= 0 || width <= 0 || vocab <= 0 || !status) return NNIS_ERR_ARGUMENT;
     int threads = width >= 256 ? 256 : 64;
     if (dtype == NNIS_DTYPE_F32)
         embed_kernel<float><<<n_tokens, threads, 0, stream>>>((const float*)table, tokens, hidden,
-                                                              n_tokens, width, vocab, status);
+                                                              n_tokens, width, vocab, status, scale);
     else if (dtype == NNIS_DTYPE_BF16)
         embed_kernel<bf16><<<n_tokens, threads, 0, stream>>>((const bf16*)table, tokens, hidden,
-                                                             n_tokens, width, vocab, status);
+                                                             n_tokens, width, vocab, status, scale);
     else
         return NNIS_ERR_UNSUPPORTED;
     NNIS_RETURN_LAUNCH();
@@ -429,8 +432,8 @@ NNIS_API int nnis_relu2_gate(const float* u, void* out, int out_dtype, long long
 
 NNIS_API int nnis_rope_part(const void* src, long long src_row, int src_head, int src_off, void* dst,
                             long long dst_row, int dst_head, int dst_off, const int* token_pos,
-                            const float* freq, int n_tokens, int heads, int len, int dims, int dtype,
-                            cudaStream_t stream) {
+                            const float* freq, int n_tokens, int heads, int len, int dims, int neighbours,
+                            int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || heads <= 0 || len <= 0 || dims < 0 || (dims & 1) || dims > len || !freq)
         return NNIS_ERR_ARGUMENT;
     int work = heads * (len - dims / 2);
@@ -439,11 +442,11 @@ NNIS_API int nnis_rope_part(const void* src, long long src_row, int src_head, in
     if (dtype == NNIS_DTYPE_F32)
         e = launch_dependent(rope_part_kernel<float>, n_tokens, threads, 0, stream, (const float*)src, src_row,
                              src_head, src_off, (float*)dst, dst_row, dst_head, dst_off, token_pos, freq, heads,
-                             len, dims);
+                             len, dims, neighbours);
     else if (dtype == NNIS_DTYPE_BF16)
         e = launch_dependent(rope_part_kernel<bf16>, n_tokens, threads, 0, stream, (const bf16*)src, src_row,
                              src_head, src_off, (bf16*)dst, dst_row, dst_head, dst_off, token_pos, freq, heads,
-                             len, dims);
+                             len, dims, neighbours);
     else
         return NNIS_ERR_UNSUPPORTED;
     return e == cudaSuccess ? NNIS_OK : (int)e;

@@ -729,20 +729,21 @@ NNIS_API int nnis_gemm_tc_act(const void* A, const void* W, const float* bias, v
 // Grouped product on the tensor cores: C[M, N] = A[M, K] . W[tile_expert[m / 128]]^T with
 // W = [experts, N, K] bfloat16 and A's rows sorted by expert in runs padded to 128 rows
 // (`tile_expert` int32 [ceil(M / 128)], negative past the last run: those tiles are left
-// alone).  The tcgen05 kernel of nnis_gemm_tc with one more coordinate for W.  `square_relu`:
-// C is bfloat16 and holds relu(.)^2; else C is float32.  Refuses (NNIS_ERR_UNSUPPORTED) K or
+// alone).  The tcgen05 kernel of nnis_gemm_tc with one more coordinate for W.  `act` (the codes of
+// nnis_gemm_tc_act): C is bfloat16 and holds act(.); 0: C is float32 and holds the sums.  Refuses (NNIS_ERR_UNSUPPORTED) K or
 // (bfloat16 C) N not a multiple of 8, (float32 C) N not a multiple of 4.
 NNIS_API int nnis_gemm_tc_grouped(const void* A, const void* W, void* C, int M, int N, int K, int experts,
-                                  const int* tile_expert, int square_relu, int sm_count, int* status, int pdl,
+                                  const int* tile_expert, int act, int sm_count, int* status, int pdl,
                                   cudaStream_t stream) {
     using namespace nnis;
     if (M <= 0 || N <= 0 || K <= 0 || experts <= 0 || !A || !W || !C || !tile_expert) return NNIS_ERR_ARGUMENT;
-    if (K % 8 || N % (square_relu ? 8 : 4) || (long long)experts * N > 0x7fffffffLL) return NNIS_ERR_UNSUPPORTED;
+    if (act < 0 || act > GEMM_ACT_GELU_TANH) return NNIS_ERR_ARGUMENT;
+    if (K % 8 || N % (act ? 8 : 4) || (long long)experts * N > 0x7fffffffLL) return NNIS_ERR_UNSUPPORTED;
     if (((uintptr_t)A | (uintptr_t)W | (uintptr_t)C) % 16) return NNIS_ERR_ALIGNMENT;
     if ((M + kBM - 1) / kBM > 65535) return NNIS_ERR_UNSUPPORTED;
     GemmArgs g = {};
     g.out = C; g.M = M; g.N = N; g.K = K; g.status = status; g.k_splits = 1;
-    g.tile_expert = tile_expert; g.expert_rows = N; g.act = square_relu ? GEMM_ACT_RELU2 : 0;
+    g.tile_expert = tile_expert; g.expert_rows = N; g.act = act;
     g.trace = trace_slot("gemm grouped");
     const int sms = sm_count > 0 ? sm_count : 148;
     const long m_tiles = (M + kBM - 1) / kBM;
@@ -750,7 +751,7 @@ NNIS_API int nnis_gemm_tc_grouped(const void* A, const void* W, void* C, int M, 
     const bool wide = tiles128 >= sms;
     CUtensorMap ma, mw, mo;
     if (!make_map(&ma, A, M, K, kBM) || !make_map(&mw, W, (long long)experts * N, K, wide ? 128 : 64) ||
-        !(square_relu ? make_map(&mo, C, M, N, kBM) : make_map(&mo, C, M, N, kBM, 0, 4)))
+        !(act ? make_map(&mo, C, M, N, kBM) : make_map(&mo, C, M, N, kBM, 0, 4)))
         return NNIS_ERR_UNSUPPORTED;
     g.out_by_tma = 1;
     const long tiles64 = m_tiles * ((N + 63) / 64);
@@ -760,7 +761,7 @@ NNIS_API int nnis_gemm_tc_grouped(const void* A, const void* W, void* C, int M, 
                                : launch_gemm_tc<128, 3, MODE, 1>(ma, mw, mo, g, pdl != 0, stream); \
     return tiles64 <= sms ? launch_gemm_tc<64, 2, MODE, 4>(ma, mw, mo, g, pdl != 0, stream) \
                           : launch_gemm_tc<64, 2, MODE, 2>(ma, mw, mo, g, pdl != 0, stream)
-    if (square_relu) { NNIS_GROUPED(GEMM_STORE); }
+    if (act) { NNIS_GROUPED(GEMM_STORE); }
     NNIS_GROUPED(GEMM_STORE_F32);
 #undef NNIS_GROUPED
 }

@@ -1,10 +1,10 @@
 // Mixture of experts, token by token: a router picks `top` of `experts` small
-// feed-forward layers W_down act(W_up h), act = relu^2, and the token's output is
-// the sum of theirs weighted by a softmax over the chosen logits only.
+// feed-forward layers W_down act(W_up h), act = relu^2 or the erf gelu, and the token's output
+// is the sum of theirs weighted by a softmax over the chosen logits only.
 //
 //   moe_route   logits z = W_r h + b in float32 (a CTA per token, a warp per expert), the `top` largest
 //               (ties to the lower index), softmax over those -> ids, weights
-//   moe_up      act[n, s, :] = relu(W_up[id[n, s]] h_n)^2: a warp per output feature
+//   moe_up      act[n, s, :] = act(W_up[id[n, s]] h_n): a warp per output feature
 //   moe_down    residual[n, :] += sum_s weight[n, s] W_down[id[n, s]] act[n, s, :], the
 //               chosen experts added in the router's order (the same bits every time)
 //
@@ -26,7 +26,9 @@
 //                     `keep` best runs can be chosen (the others' c counts as minus infinity); the `top`
 //                     largest c (ties to the lower index) are chosen and weighed by their s as it is.
 //                     Outputs from `experts` on have no matrices: their id is written as -1 and their
-//                     weights are added up in `pass_weight[n]`
+//                     weights are added up in `pass_weight[n]`.  Options: scores sigmoid(z) output by
+//                     output instead of the softmax; a run's score the sum of its two largest c (of its
+//                     one c, where a run has one output); the chosen weights divided by their sum + 1e-20
 //   moe_up_gated      with no weights: act = silu(g) * u; a pair whose id is negative is skipped
 //   moe_down          with weights on the outputs, skipping negative ids, plus pass_weight[n] * h[n]
 //
@@ -151,7 +153,7 @@ __global__ void __launch_bounds__(256)
 moe_route_choice_kernel(const T* __restrict__ h, const float* __restrict__ wr, const float* __restrict__ correction,
                         const int* __restrict__ token_pos, int* __restrict__ ids, float* __restrict__ weights,
                         float* __restrict__ pass_weight, int n_tokens, int width, int outputs, int experts, int top,
-                        int groups, int keep) {
+                        int groups, int keep, int sigmoid_scores, int group_top, int renormalise) {
     extern __shared__ float z_all[];
     const int per = 2 * outputs + groups;
     pdl_wait();
@@ -244,30 +246,41 @@ moe_route_choice_kernel(const T* __restrict__ h, const float* __restrict__ wr, c
         if (lane == 0) pass_weight[n] = 0.f;
         return;
     }
-    // one softmax over all outputs
-    float mx = -FLT_MAX;
-    for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, z[e]);
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int e = lane; e < outputs; e += 32) {
-        const float p = expf(z[e] - mx);
-        z[e] = p;
-        sum += p;
-    }
-    sum = warp_sum(sum);
-    const float inv = 1.0f / sum;
-    for (int e = lane; e < outputs; e += 32) {
-        const float s = z[e] * inv;
-        z[e] = s;
-        choice[e] = s + (correction ? correction[e] : 0.f);
+    if (sigmoid_scores) {
+        for (int e = lane; e < outputs; e += 32) {
+            const float s = 1.0f / (1.0f + expf(-z[e]));
+            z[e] = s;
+            choice[e] = s + (correction ? correction[e] : 0.f);
+        }
+    } else {  // one softmax over all outputs
+        float mx = -FLT_MAX;
+        for (int e = lane; e < outputs; e += 32) mx = fmaxf(mx, z[e]);
+        mx = warp_max(mx);
+        float sum = 0.f;
+        for (int e = lane; e < outputs; e += 32) {
+            const float p = expf(z[e] - mx);
+            z[e] = p;
+            sum += p;
+        }
+        sum = warp_sum(sum);
+        const float inv = 1.0f / sum;
+        for (int e = lane; e < outputs; e += 32) {
+            const float s = z[e] * inv;
+            z[e] = s;
+            choice[e] = s + (correction ? correction[e] : 0.f);
+        }
     }
     __syncwarp();
     if (groups > 1 && keep < groups) {
         const int size = outputs / groups;
         for (int g = lane; g < groups; g += 32) {
-            float best = -INFINITY;
-            for (int e = g * size; e < (g + 1) * size; ++e) best = fmaxf(best, choice[e]);
-            run_best[g] = best;
+            float best = -INFINITY, second = -INFINITY;
+            for (int e = g * size; e < (g + 1) * size; ++e) {
+                const float v = choice[e];
+                second = fmaxf(second, fminf(best, v));
+                best = fmaxf(best, v);
+            }
+            run_best[g] = (group_top == 2 && size > 1) ? best + second : best;
         }
         __syncwarp();
         // the runs that are NOT among the `keep` best: a run is kept if fewer than `keep` runs beat it
@@ -281,7 +294,7 @@ moe_route_choice_kernel(const T* __restrict__ h, const float* __restrict__ wr, c
         }
         __syncwarp();
     }
-    float passed = 0.f;
+    float passed = 0.f, total = 0.f;
     for (int s = 0; s < top; ++s) {
         float best = -INFINITY;
         int arg = 0x7fffffff;
@@ -302,6 +315,7 @@ moe_route_choice_kernel(const T* __restrict__ h, const float* __restrict__ wr, c
             }
         }
         const float score = z[arg];
+        total += score;
         if (arg >= experts) passed += score;
         __syncwarp();
         if (lane == 0) {
@@ -312,27 +326,36 @@ moe_route_choice_kernel(const T* __restrict__ h, const float* __restrict__ wr, c
         }
         __syncwarp();
     }
+    if (renormalise) {
+        const float inv = 1.0f / (total + 1e-20f);
+        for (int s = lane; s < top; s += 32) wt[s] *= inv;
+        passed *= inv;
+    }
     if (lane == 0) pass_weight[n] = passed;
+}
+
+// the experts' activations, by the codes of the storing products' epilogues: 1 relu(x)^2, 2 gelu with erf
+__device__ __forceinline__ float expert_act(float x, int act) {
+    if (act == 2) return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f));
+    const float a = fmaxf(x, 0.f);
+    return a * a;
 }
 
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_up_kernel(const T* __restrict__ h, const T* __restrict__ w_up, const int* __restrict__ ids,
-              const int* __restrict__ token_pos, T* __restrict__ act, int width, int ff, int top) {
+              const int* __restrict__ token_pos, T* __restrict__ act, int width, int ff, int top, int act_kind) {
     pdl_wait();
     pdl_launch_dependents();
     int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     long long pair = blockIdx.x;
     int f = blockIdx.y * 8 + warp;
     long long n = pair / top;
-    if (f >= ff || token_pos[n] < 0) return;
+    if (f >= ff || token_pos[n] < 0 || ids[pair] < 0) return;
     const T* w = w_up + ((size_t)ids[pair] * ff + f) * width;
     const T* x = h + (size_t)n * width;
     float acc = warp_row_dot(w, x, width, lane);
-    if (lane == 0) {
-        float a = fmaxf(acc, 0.f);
-        act[(size_t)pair * ff + f] = from_float<T>(a * a);
-    }
+    if (lane == 0) act[(size_t)pair * ff + f] = from_float<T>(expert_act(acc, act_kind));
 }
 
 template <typename T>
@@ -409,13 +432,15 @@ NNIS_API int nnis_moe_route(const void* h, const float* wr, const float* br, con
     return e == cudaSuccess ? NNIS_OK : (int)e;
 }
 
-// act: operand dtype [n_tokens, top, ff] (scratch); residual: float32 [n_tokens, width]
+// act: operand dtype [n_tokens, top, ff] (scratch); residual: float32 [n_tokens, width]; act_kind: 1
+// relu^2, 2 gelu with erf; a pair with a negative id has no expert; pass_weight (float32 [n_tokens] or
+// null) times the token's input is added
 NNIS_API int nnis_moe_experts(const void* h, const void* w_up, const void* w_down, const int* ids,
-                              const float* weights, const int* token_pos, void* act, float* residual,
-                              int n_tokens, int width, int ff, int top, int dtype,
+                              const float* weights, const float* pass_weight, const int* token_pos, void* act,
+                              float* residual, int n_tokens, int width, int ff, int top, int act_kind, int dtype,
                               cudaStream_t stream) {
     if (n_tokens <= 0 || width <= 0 || ff <= 0 || top <= 0 || !h || !w_up || !w_down || !ids ||
-        !weights || !token_pos || !act || !residual)
+        !weights || !token_pos || !act || !residual || (act_kind != 1 && act_kind != 2))
         return NNIS_ERR_ARGUMENT;
     if ((ff + 7) / 8 > 65535 || (width + 7) / 8 > 65535) return NNIS_ERR_UNSUPPORTED;
     dim3 up_grid((unsigned)((long long)n_tokens * top), (ff + 7) / 8);
@@ -423,16 +448,18 @@ NNIS_API int nnis_moe_experts(const void* h, const void* w_up, const void* w_dow
     cudaError_t e;
     if (dtype == NNIS_DTYPE_F32) {
         e = launch_dependent(moe_up_kernel<float>, up_grid, 256, 0, stream, (const float*)h, (const float*)w_up, ids,
-                             token_pos, (float*)act, width, ff, top);
+                             token_pos, (float*)act, width, ff, top, act_kind);
         if (e == cudaSuccess)
             e = launch_dependent(moe_down_kernel<float>, down_grid, 256, 0, stream, (const float*)act,
-                                 (const float*)w_down, ids, weights, token_pos, residual, width, ff, top, (const float*)nullptr, (const float*)nullptr);
+                                 (const float*)w_down, ids, weights, token_pos, residual, width, ff, top, pass_weight,
+                                 (const float*)h);
     } else if (dtype == NNIS_DTYPE_BF16) {
         e = launch_dependent(moe_up_kernel<bf16>, up_grid, 256, 0, stream, (const bf16*)h, (const bf16*)w_up, ids,
-                             token_pos, (bf16*)act, width, ff, top);
+                             token_pos, (bf16*)act, width, ff, top, act_kind);
         if (e == cudaSuccess)
             e = launch_dependent(moe_down_kernel<bf16>, down_grid, 256, 0, stream, (const bf16*)act,
-                                 (const bf16*)w_down, ids, weights, token_pos, residual, width, ff, top, (const float*)nullptr, (const bf16*)nullptr);
+                                 (const bf16*)w_down, ids, weights, token_pos, residual, width, ff, top, pass_weight,
+                                 (const bf16*)h);
     } else {
         return NNIS_ERR_UNSUPPORTED;
     }
@@ -473,14 +500,15 @@ NNIS_API int nnis_moe_experts_gated(const void* h, const void* w_gu, const void*
 
 // The router that scores all its outputs with one softmax: see moe_route_choice above.  wr float32
 // [outputs, width]; correction float32 [outputs] or null; ids int32 [n, top] (-1: an output from
-// `experts` on); weights float32 [n, top]; pass_weight float32 [n].
+// `experts` on); weights float32 [n, top]; pass_weight float32 [n]; sigmoid_scores, group_top (1 or 2),
+// renormalise: the options named there.
 NNIS_API int nnis_moe_route_choice(const void* h, const float* wr, const float* correction, const int* token_pos,
                                    int* ids, float* weights, float* pass_weight, int n_tokens, int width,
-                                   int outputs, int experts, int top, int groups, int keep, int dtype,
-                                   cudaStream_t stream) {
+                                   int outputs, int experts, int top, int groups, int keep, int sigmoid_scores,
+                                   int group_top, int renormalise, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || width <= 0 || outputs <= 0 || experts < 0 || experts > outputs || top <= 0 ||
         top > outputs || groups <= 0 || outputs % groups || keep <= 0 || keep > groups || !h || !wr || !ids ||
-        !weights || !pass_weight || !token_pos)
+        !weights || !pass_weight || !token_pos || (group_top != 1 && group_top != 2))
         return NNIS_ERR_ARGUMENT;
     if (top > keep * (outputs / groups)) return NNIS_ERR_ARGUMENT;
     const size_t per = (2 * (size_t)outputs + groups) * sizeof(float);
@@ -492,7 +520,8 @@ NNIS_API int nnis_moe_route_choice(const void* h, const float* wr, const float* 
     cudaError_t e;
 #define NNIS_ROUTE(T, TOK) \
     launch_dependent(moe_route_choice_kernel<T, TOK>, blocks, 256, smem, stream, (const T*)h, wr, correction, \
-                     token_pos, ids, weights, pass_weight, n_tokens, width, outputs, experts, top, groups, keep)
+                     token_pos, ids, weights, pass_weight, n_tokens, width, outputs, experts, top, groups, keep, \
+                     sigmoid_scores, group_top, renormalise)
     if (dtype == NNIS_DTYPE_F32)
         e = several ? NNIS_ROUTE(float, 4) : NNIS_ROUTE(float, 1);
     else if (dtype == NNIS_DTYPE_BF16)

@@ -8,7 +8,8 @@
 //   grouped_mma   C[tile rows, N] = A[rows] . W[expert]^T: 64 x 64 tiles, K in slices of 64
 //                 through a three-stage cp.async ring into swizzled shared memory,
 //                 mma.sync m16n8k16, float32 accumulation.  The first product gathers its
-//                 rows from the tokens' inputs by `perm` and stores relu^2 in bfloat16; the
+//                 rows from the tokens' inputs by `perm` and stores the activation (relu^2 or the
+//                 erf gelu) in bfloat16; the
 //                 second reads the sorted activations and stores float32.
 //   moe_combine   residual[n] += sum_s weight[n, s] * y[place[n, s]], in the router's order
 //
@@ -20,7 +21,7 @@
 // Where an expert gets many rows (nnis_moe_grouped_tc) the runs are padded to 128 rows
 // instead, moe_gather puts the tokens' inputs into the sorted order, and both products run
 // on the tcgen05 kernel of the dense projections with one weight matrix per tile of rows
-// (gemm_tcgen05.cu: nnis_gemm_tc_grouped), relu^2 in the first one's epilogue.
+// (gemm_tcgen05.cu: nnis_gemm_tc_grouped), the activation in the first one's epilogue.
 //
 // A row's result depends on nothing but the row, so the order inside an expert's run
 // (which the sort's atomics decide) changes no bit of the output.
@@ -78,7 +79,7 @@ moe_sort_kernel(const int* __restrict__ ids, int n_pairs, int experts, int max_t
     }
 }
 
-// MODE 0: rows gathered from x by perm (pair / top), epilogue relu^2 -> bfloat16
+// MODE 0: rows gathered from x by perm (pair / top), epilogue relu^2 (act 1) or gelu (2) -> bfloat16
 // MODE 1: rows of a in sorted order, epilogue float32
 // MODE 2: one matrix per head (blockIdx.z) on packed rows: rows 0 .. M - 1 of a, the head's
 //         slice a_bs apart in a and c_bs apart in out (row stride ldc), bfloat16 out
@@ -87,7 +88,7 @@ __global__ void __launch_bounds__(128)
 grouped_mma_kernel(const bf16* __restrict__ a, int lda, const int* __restrict__ perm, int top,
                    const bf16* __restrict__ w, const int* __restrict__ tile_expert,
                    void* __restrict__ out, int N, int K, int M, long long a_bs, int ldc,
-                   long long c_bs, const float* __restrict__ pair_weight = nullptr) {
+                   long long c_bs, const float* __restrict__ pair_weight = nullptr, int act = 1) {
     constexpr int BK = 64, STAGES = 3, CH = BK / 8;
     const int expert = MODE == 2 ? (int)blockIdx.z : tile_expert[blockIdx.x];
     if (expert < 0) return;
@@ -174,11 +175,18 @@ grouped_mma_kernel(const bf16* __restrict__ a, int lda, const int* __restrict__ 
                 if (col + 1 < N) o[(size_t)(row0 + r) * (N >> 1) + (col >> 1)] =
                     __float2bfloat16_rn(g / (1.0f + __expf(-g)) * u);
             } else if (MODE == 0) {
-                v0 = fmaxf(v0, 0.f);
-                v1 = fmaxf(v1, 0.f);
+                if (act == 2) {
+                    v0 = 0.5f * v0 * (1.0f + erff(v0 * 0.70710678118654752f));
+                    v1 = 0.5f * v1 * (1.0f + erff(v1 * 0.70710678118654752f));
+                } else {
+                    v0 = fmaxf(v0, 0.f);
+                    v1 = fmaxf(v1, 0.f);
+                    v0 *= v0;
+                    v1 *= v1;
+                }
                 bf16* o = reinterpret_cast<bf16*>(out);
-                if (col < N) o[base + col] = __float2bfloat16_rn(v0 * v0);
-                if (col + 1 < N) o[base + col + 1] = __float2bfloat16_rn(v1 * v1);
+                if (col < N) o[base + col] = __float2bfloat16_rn(v0);
+                if (col + 1 < N) o[base + col + 1] = __float2bfloat16_rn(v1);
             } else {
                 float* o = reinterpret_cast<float*>(out);
                 if (col < N) o[base + col] = v0;
@@ -294,13 +302,15 @@ NNIS_API int nnis_moe_grouped_takes(int width, int ff, int experts) {
 // x: bfloat16 [n_tokens, width]; ids, weights [n_tokens, top] from the router (every row a
 // token: no padding rows); scratch: perm int32 [tiles * 64], place int32 [n_tokens * top],
 // tile_expert int32 [tiles], act bfloat16 [tiles * 64, ff], y float32 [tiles * 64, width]
-// with tiles = nnis_moe_grouped_tiles(n_tokens * top, experts).
+// with tiles = nnis_moe_grouped_tiles(n_tokens * top, experts); act_kind: 1 relu^2, 2 gelu with erf;
+// a pair with a negative id has no expert; pass_weight (float32 [n_tokens] or null) times the token's
+// input is added.
 NNIS_API int nnis_moe_grouped(const void* x, const void* w_up, const void* w_down, const int* ids,
                               const float* weights, int* perm, int* place, int* tile_expert, void* act,
                               float* y, float* residual, int n_tokens, int width, int ff, int experts,
-                              int top, cudaStream_t stream) {
+                              int top, int act_kind, const float* pass_weight, cudaStream_t stream) {
     if (n_tokens <= 0 || top <= 0 || !x || !w_up || !w_down || !ids || !weights || !perm || !place ||
-        !tile_expert || !act || !y || !residual)
+        !tile_expert || !act || !y || !residual || (act_kind != 1 && act_kind != 2))
         return NNIS_ERR_ARGUMENT;
     if (!nnis_moe_grouped_takes(width, ff, experts)) return NNIS_ERR_UNSUPPORTED;
     if (((uintptr_t)x | (uintptr_t)w_up | (uintptr_t)w_down | (uintptr_t)act) % 16) return NNIS_ERR_ALIGNMENT;
@@ -312,11 +322,12 @@ NNIS_API int nnis_moe_grouped(const void* x, const void* w_up, const void* w_dow
     int code = configure_grouped();
     if (code != NNIS_OK) return code;
     grouped_mma_kernel<0><<<dim3(tiles, (ff + 63) / 64), 128, smem, stream>>>(
-        (const bf16*)x, width, perm, top, (const bf16*)w_up, tile_expert, act, ff, width, 0, 0, 0, 0);
+        (const bf16*)x, width, perm, top, (const bf16*)w_up, tile_expert, act, ff, width, 0, 0, 0, 0,
+        (const float*)nullptr, act_kind);
     grouped_mma_kernel<1><<<dim3(tiles, (width + 63) / 64), 128, smem, stream>>>(
         (const bf16*)act, ff, perm, top, (const bf16*)w_down, tile_expert, y, width, ff, 0, 0, 0, 0);
-    moe_combine_kernel<<<n_tokens, 256, 0, stream>>>(y, place, weights, residual, width, top,
-                                                     (const float*)nullptr, (const bf16*)nullptr);
+    moe_combine_kernel<<<n_tokens, 256, 0, stream>>>(y, place, weights, residual, width, top, pass_weight,
+                                                     (const bf16*)x);
     NNIS_RETURN_LAUNCH();
 }
 
@@ -352,23 +363,24 @@ NNIS_API int nnis_moe_grouped_gated(const void* x, const void* w_gu, const void*
 }
 
 // The same with both products on the tcgen05 kernel (nnis_gemm_tc_grouped): runs padded to
-// 128 rows, the first product's rows gathered into x_sorted [tiles * 128, width] first, relu^2
-// in that product's epilogue.  tiles = nnis_moe_grouped_tiles_tc(n_tokens * top, experts);
+// 128 rows, the first product's rows gathered into x_sorted [tiles * 128, width] first, the
+// activation in that product's epilogue.  tiles = nnis_moe_grouped_tiles_tc(n_tokens * top, experts);
 // scratch as nnis_moe_grouped with 128 rows a tile, plus x_sorted (bfloat16).
 NNIS_API int nnis_moe_grouped_tiles_tc(long long n_pairs, int experts) {
     return (int)((n_pairs + 127) / 128) + experts;
 }
 
 extern "C" int nnis_gemm_tc_grouped(const void* A, const void* W, void* C, int M, int N, int K, int experts,
-                                    const int* tile_expert, int square_relu, int sm_count, int* status, int pdl,
+                                    const int* tile_expert, int act, int sm_count, int* status, int pdl,
                                     cudaStream_t stream);
 
 NNIS_API int nnis_moe_grouped_tc(const void* x, const void* w_up, const void* w_down, const int* ids,
                                  const float* weights, int* perm, int* place, int* tile_expert, void* x_sorted,
                                  void* act, float* y, float* residual, int n_tokens, int width, int ff,
-                                 int experts, int top, int sm_count, int* status, int pdl, cudaStream_t stream) {
+                                 int experts, int top, int act_kind, const float* pass_weight, int sm_count,
+                                 int* status, int pdl, cudaStream_t stream) {
     if (n_tokens <= 0 || top <= 0 || !x || !w_up || !w_down || !ids || !weights || !perm || !place ||
-        !tile_expert || !x_sorted || !act || !y || !residual)
+        !tile_expert || !x_sorted || !act || !y || !residual || (act_kind != 1 && act_kind != 2))
         return NNIS_ERR_ARGUMENT;
     if (!nnis_moe_grouped_takes(width, ff, experts)) return NNIS_ERR_UNSUPPORTED;
     if (((uintptr_t)x | (uintptr_t)x_sorted) % 16) return NNIS_ERR_ALIGNMENT;
@@ -380,14 +392,14 @@ NNIS_API int nnis_moe_grouped_tc(const void* x, const void* w_up, const void* w_
     cudaError_t e = launch_dependent(moe_gather_kernel, (unsigned)rows, 256, 0, stream, (const bf16*)x,
                                      (const int*)perm, top, (bf16*)x_sorted, width);
     if (e != cudaSuccess) return (int)e;
-    int code = nnis_gemm_tc_grouped(x_sorted, w_up, act, rows, ff, width, experts, tile_expert, 1, sm_count, status,
+    int code = nnis_gemm_tc_grouped(x_sorted, w_up, act, rows, ff, width, experts, tile_expert, act_kind, sm_count, status,
                                     pdl, stream);
     if (code != NNIS_OK) return code;
     code = nnis_gemm_tc_grouped(act, w_down, y, rows, width, ff, experts, tile_expert, 0, sm_count, status, pdl,
                                 stream);
     if (code != NNIS_OK) return code;
-    moe_combine_kernel<<<n_tokens, 256, 0, stream>>>(y, place, weights, residual, width, top,
-                                                     (const float*)nullptr, (const bf16*)nullptr);
+    moe_combine_kernel<<<n_tokens, 256, 0, stream>>>(y, place, weights, residual, width, top, pass_weight,
+                                                     (const bf16*)x);
     NNIS_RETURN_LAUNCH();
 }
 

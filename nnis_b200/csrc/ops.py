@@ -81,8 +81,8 @@ def code_of(dtype: torch.dtype) -> int:
 
 # ---------------------------------------------------------------------------
 def embed(table: torch.Tensor, tokens: torch.Tensor, hidden: torch.Tensor,
-          status: torch.Tensor) -> None:
-    """hidden[n] = table[tokens[n]] widened to float32; an id outside the table
+          status: torch.Tensor, scale: float = 1.0) -> None:
+    """hidden[n] = table[tokens[n]] widened to float32, times ``scale``; an id outside the table
     sets ``status[0]`` and yields a zero row."""
     _cuda(table, tokens, hidden, status)
     n, width = hidden.shape
@@ -90,7 +90,7 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, hidden: torch.Tensor,
     _need(hidden.dtype == torch.float32 and table.shape[1] == width, "hidden: float32 [n, width]")
     _need(status.dtype == torch.int32, "status: int32")
     _check(_lib().nnis_embed(_ptr(table), code_of(table.dtype), _ptr(tokens), _ptr(hidden), n, width,
-                             table.shape[0], _ptr(status), _stream()), "embed")
+                             table.shape[0], _ptr(status), ctypes.c_float(scale), _stream()), "embed")
 
 
 def copy_async(dst: torch.Tensor, src: torch.Tensor) -> None:
@@ -1007,10 +1007,12 @@ def relu2_gate(u: torch.Tensor, out: torch.Tensor) -> None:
 
 def rope_part(src: torch.Tensor, src_head: int, src_off: int, dst: torch.Tensor, dst_head: int,
               dst_off: int, token_pos: torch.Tensor, freq: torch.Tensor, heads: int, length: int,
-              dims: int) -> None:
+              dims: int, pairing: str = "half") -> None:
     """For every row n and head h, the ``length`` elements at src[n, h * src_head + src_off]
     go to dst[n, h * dst_head + dst_off]; the first ``dims`` are turned in pairs (i, i +
-    dims / 2) by the angle position * freq[i], the rest pass unchanged."""
+    dims / 2), or with ``pairing`` "neighbours" (2i, 2i + 1), by the angle position * freq[i],
+    the rest pass unchanged."""
+    _need(pairing in ("neighbours", "half"), "rope_part: pairing is neighbours or half")
     _cuda(src, dst, token_pos, freq)
     n = src.shape[0]
     _need(src.dtype == dst.dtype and dst.shape[0] == n, "rope_part: src and dst of one dtype and row count")
@@ -1023,7 +1025,8 @@ def rope_part(src: torch.Tensor, src_head: int, src_off: int, dst: torch.Tensor,
     _need(token_pos.dtype == torch.int32 and token_pos.numel() >= n, "rope_part: token_pos int32 [n]")
     _check(_lib().nnis_rope_part(_ptr(src), ctypes.c_longlong(src.shape[1]), src_head, src_off, _ptr(dst),
                                  ctypes.c_longlong(dst.shape[1]), dst_head, dst_off, _ptr(token_pos),
-                                 _ptr(freq), n, heads, length, dims, code_of(src.dtype), _stream()),
+                                 _ptr(freq), n, heads, length, dims, 1 if pairing == "neighbours" else 0,
+                                 code_of(src.dtype), _stream()),
            "rope_part")
 
 
@@ -1054,9 +1057,10 @@ def batched_linear(a: torch.Tensor, a_head: int, w: torch.Tensor, out: torch.Ten
 def latent_prep(a: torch.Tensor, wq: torch.Tensor, wkv: torch.Tensor, freq: torch.Tensor,
                 token_pos: torch.Tensor, token_seq: torch.Tensor, page_table: torch.Tensor,
                 cq: torch.Tensor, cache: torch.Tensor, q_rank: int, kv_rank: int, rot: int,
-                rot_dims: int, eps: float) -> None:
+                rot_dims: int, eps: float, pairing: str = "half") -> None:
     """From the down-projection's float32 rows [q latent | c raw | kr raw]: the normed q
     latent to ``cq``; the normed c and the rotated kr into the cache row of each token."""
+    _need(pairing in ("neighbours", "half"), "latent_prep: pairing is neighbours or half")
     _cuda(a, wq, wkv, freq, token_pos, token_seq, page_table, cq, cache)
     n = a.shape[0]
     _need(a.dtype == torch.float32 and a.shape[1] == q_rank + kv_rank + rot, "latent_prep: a float32 rows")
@@ -1069,16 +1073,50 @@ def latent_prep(a: torch.Tensor, wq: torch.Tensor, wkv: torch.Tensor, freq: torc
     _check(_lib().nnis_latent_prep(_ptr(a), _ptr(wq), _ptr(wkv), _ptr(freq), _ptr(token_pos),
                                    _ptr(token_seq), _ptr(page_table), page_table.shape[1], _ptr(cq),
                                    _ptr(cache), n, q_rank, kv_rank, rot, rot_dims, cache.shape[2],
-                                   ctypes.c_float(eps), code_of(cq.dtype), _stream()), "latent_prep")
+                                   ctypes.c_float(eps), 1 if pairing == "neighbours" else 0, code_of(cq.dtype),
+                                   _stream()), "latent_prep")
+
+
+def latent_prep_direct(a: torch.Tensor, wkv: torch.Tensor, freq: torch.Tensor, token_pos: torch.Tensor,
+                       token_seq: torch.Tensor, page_table: torch.Tensor, q_plain: torch.Tensor,
+                       q_rows: torch.Tensor, cache: torch.Tensor, gate: Optional[torch.Tensor], heads: int, dim: int,
+                       kv_rank: int, rot: int, rot_dims: int, eps: float, pairing: str = "half") -> None:
+    """From float32 rows [q (heads x (dim plain | rot rotated)) | c raw | kr raw | gate logits]: the plain
+    parts of q packed to ``q_plain`` [n, heads * dim], the rotated ones turned into the last ``rot``
+    values of every head of ``q_rows`` [n, heads * (kv_rank + rot)], the normed c and the turned kr
+    into the cache row of each token, and the sigmoid of the gate's logits (``gate`` [n, heads] or None)."""
+    _cuda(a, wkv, freq, token_pos, token_seq, page_table, q_plain, q_rows, cache, gate)
+    n = a.shape[0]
+    _need(pairing in ("neighbours", "half"), "latent_prep_direct: pairing is neighbours or half")
+    _need(a.dtype == torch.float32 and a.shape[1] >= heads * (dim + rot) + kv_rank + rot + (heads if gate is not None else 0),
+          "latent_prep_direct: a float32 rows (further columns are padding)")
+    _need(wkv.dtype == freq.dtype == torch.float32 and wkv.numel() == kv_rank and freq.numel() >= rot_dims // 2,
+          "latent_prep_direct: float32 vectors")
+    _need(q_plain.dtype == q_rows.dtype == cache.dtype and tuple(q_plain.shape) == (n, heads * dim)
+          and tuple(q_rows.shape) == (n, heads * (kv_rank + rot)), "latent_prep_direct: q_plain, q_rows")
+    _need(cache.dim() == 4 and cache.shape[1] == 1 and cache.shape[3] == kv_rank + rot,
+          "latent_prep_direct: cache [pages, 1, page, kv_rank + rot]")
+    _need(gate is None or (gate.dtype == torch.float32 and tuple(gate.shape) == (n, heads)),
+          "latent_prep_direct: gate float32 [n, heads]")
+    _need(page_table.dtype == torch.int32 and token_pos.dtype == torch.int32, "latent_prep_direct: int32 tables")
+    _check(_lib().nnis_latent_prep_direct(_ptr(a), _ptr(wkv), _ptr(freq), _ptr(token_pos), _ptr(token_seq),
+                                          _ptr(page_table), page_table.shape[1], _ptr(q_plain), _ptr(q_rows),
+                                          _ptr(cache), _ptr(gate), n, heads, dim, kv_rank, rot, rot_dims,
+                                          cache.shape[2], ctypes.c_float(eps), 1 if pairing == "neighbours" else 0,
+                                          a.shape[1], code_of(q_plain.dtype), _stream()), "latent_prep_direct")
 
 
 def attention_latent(q: torch.Tensor, cache: torch.Tensor, token_pos: torch.Tensor,
                      token_seq: torch.Tensor, page_table: torch.Tensor, out: torch.Tensor, heads: int,
                      dv: int, scale: float, n_splits: int = 1,
-                     partial: Optional[torch.Tensor] = None) -> None:
+                     partial: Optional[torch.Tensor] = None, window: int = 0,
+                     gate: Optional[torch.Tensor] = None) -> None:
     """Causal attention of packed queries [n, heads * dk] over cache rows [pages, 1, page,
-    dk] shared by all heads; the rows' first ``dv`` values are the values.  out [n, heads * dv]."""
-    _cuda(q, cache, token_pos, token_seq, page_table, out, partial)
+    dk] shared by all heads; the rows' first ``dv`` values are the values.  out [n, heads * dv].
+    ``window`` > 0: a query sees that many keys, itself included; ``gate`` (float32 [n, heads])
+    multiplies each head's output."""
+    _cuda(q, cache, token_pos, token_seq, page_table, out, partial, gate)
+    _need(gate is None or (gate.dtype == torch.float32 and gate.numel() >= out.shape[0] * heads), "attention_latent: gate")
     n = out.shape[0]
     pages, one, page_size, dk = cache.shape
     _need(one == 1 and q.shape[1] == heads * dk and out.shape[1] == heads * dv and 0 < dv <= dk,
@@ -1090,8 +1128,8 @@ def attention_latent(q: torch.Tensor, cache: torch.Tensor, token_pos: torch.Tens
               and partial.numel() >= n * heads * n_splits * (dv + 2), "attention_latent: partial scratch")
     _check(_lib().nnis_attention_latent(_ptr(q), _ptr(cache), _ptr(token_pos), _ptr(token_seq),
                                         _ptr(page_table), page_table.shape[1], _ptr(out), _ptr(partial), n,
-                                        heads, dk, dv, page_size, ctypes.c_float(scale), n_splits,
-                                        code_of(out.dtype), _stream()),
+                                        heads, dk, dv, page_size, ctypes.c_float(scale), n_splits, window,
+                                        _ptr(gate), code_of(out.dtype), _stream()),
            "attention_latent", 2 if n_splits > 1 else 1)
 
 
@@ -1184,17 +1222,19 @@ def moe_route(h: torch.Tensor, w_router: torch.Tensor, b_router: Optional[torch.
 
 def moe_experts(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
                 weights: torch.Tensor, token_pos: torch.Tensor, act: torch.Tensor,
-                residual: torch.Tensor, top: int) -> None:
-    """residual[n] += sum over the chosen experts of weight * W_down[e] relu(W_up[e] h[n])^2."""
-    _cuda(h, w_up, w_down, ids, weights, token_pos, act, residual)
+                residual: torch.Tensor, top: int, activation: int = GEMM_ACT_RELU2,
+                pass_weight: Optional[torch.Tensor] = None) -> None:
+    """residual[n] += sum over the chosen experts of weight * W_down[e] act(W_up[e] h[n]), act the square
+    of relu or (``GEMM_ACT_GELU_ERF``) the erf gelu, + pass_weight[n] * h[n]; a negative id has no expert."""
+    _cuda(h, w_up, w_down, ids, weights, token_pos, act, residual, pass_weight)
     n, width = h.shape
     experts, ff, _ = w_up.shape
     _need(tuple(w_up.shape) == (experts, ff, width) and tuple(w_down.shape) == (experts, width, ff)
           and h.dtype == w_up.dtype == w_down.dtype == act.dtype, "moe_experts: stacked weights of one dtype")
     _need(act.numel() >= n * top * ff, "moe_experts: act scratch [n, top, ff]")
     _need(residual.dtype == torch.float32 and tuple(residual.shape) == (n, width), "moe_experts: residual")
-    _check(_lib().nnis_moe_experts(_ptr(h), _ptr(w_up), _ptr(w_down), _ptr(ids), _ptr(weights),
-                                   _ptr(token_pos), _ptr(act), _ptr(residual), n, width, ff, top,
+    _check(_lib().nnis_moe_experts(_ptr(h), _ptr(w_up), _ptr(w_down), _ptr(ids), _ptr(weights), _ptr(pass_weight),
+                                   _ptr(token_pos), _ptr(act), _ptr(residual), n, width, ff, top, activation,
                                    code_of(h.dtype), _stream()), "moe_experts", 2)
 
 
@@ -1226,11 +1266,13 @@ def attention_latent_mma(q: torch.Tensor, cache: torch.Tensor, tiles: Optional[t
                          seq_first_row: Optional[torch.Tensor], seq_start: Optional[torch.Tensor],
                          seq_count: Optional[torch.Tensor], token_pos: torch.Tensor, token_seq: torch.Tensor,
                          page_table: torch.Tensor, out: torch.Tensor, heads: int, dv: int, scale: float,
-                         n_splits: int = 1, partial: Optional[torch.Tensor] = None) -> None:
+                         n_splits: int = 1, partial: Optional[torch.Tensor] = None, window: int = 0,
+                         gate: Optional[torch.Tensor] = None) -> None:
     """``attention_latent`` on the tensor cores (bfloat16).  With ``tiles`` (``latent_tiles``) a
     prompt step; without, every row is one token of a sequence of its own."""
-    _cuda(q, cache, tiles, seq_first_row, seq_start, seq_count, token_pos, token_seq, page_table, out, partial)
+    _cuda(q, cache, tiles, seq_first_row, seq_start, seq_count, token_pos, token_seq, page_table, out, partial, gate)
     n = out.shape[0]
+    _need(gate is None or (gate.dtype == torch.float32 and gate.numel() >= n * heads), "attention_latent_mma: gate")
     pages, one, page_size, dk = cache.shape
     _need(q.dtype == cache.dtype == out.dtype == torch.bfloat16, "attention_latent_mma: bfloat16")
     _need(one == 1 and q.shape[1] == heads * dk and out.shape[1] == heads * dv, "attention_latent_mma: shapes")
@@ -1243,7 +1285,7 @@ def attention_latent_mma(q: torch.Tensor, cache: torch.Tensor, tiles: Optional[t
         _ptr(q), _ptr(cache), _ptr(tiles), tiles.shape[0] if tiles is not None else 0, _ptr(seq_first_row),
         _ptr(seq_start), _ptr(seq_count), _ptr(token_pos), _ptr(token_seq), _ptr(page_table),
         page_table.shape[1], _ptr(out), _ptr(partial), n, heads, dk, dv, page_size, ctypes.c_float(scale),
-        n_splits, _stream()), "attention_latent_mma", 2 if n_splits > 1 else 1)
+        n_splits, window, _ptr(gate), _stream()), "attention_latent_mma", 2 if n_splits > 1 else 1)
 
 
 
@@ -1259,11 +1301,12 @@ def moe_grouped_tiles(n_pairs: int, experts: int) -> int:
 
 def moe_grouped(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
                 weights: torch.Tensor, perm: torch.Tensor, place: torch.Tensor, tile_expert: torch.Tensor,
-                act: torch.Tensor, y: torch.Tensor, residual: torch.Tensor, top: int) -> None:
+                act: torch.Tensor, y: torch.Tensor, residual: torch.Tensor, top: int,
+                activation: int = GEMM_ACT_RELU2, pass_weight: Optional[torch.Tensor] = None) -> None:
     """``moe_experts`` for many tokens: pairs sorted by expert, two grouped products on the
     tensor cores, the chosen experts' outputs added in the router's order.  Every row of
     ``h`` is a token (no padding rows).  Scratch sizes: see ``moe_grouped_tiles``."""
-    _cuda(h, w_up, w_down, ids, weights, perm, place, tile_expert, act, y, residual)
+    _cuda(h, w_up, w_down, ids, weights, perm, place, tile_expert, act, y, residual, pass_weight)
     n, width = h.shape
     experts, ff, _ = w_up.shape
     tiles = moe_grouped_tiles(n * top, experts)
@@ -1279,7 +1322,7 @@ def moe_grouped(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: 
     _need(residual.dtype == torch.float32 and tuple(residual.shape) == (n, width), "moe_grouped: residual")
     _check(_lib().nnis_moe_grouped(_ptr(h), _ptr(w_up), _ptr(w_down), _ptr(ids), _ptr(weights), _ptr(perm),
                                    _ptr(place), _ptr(tile_expert), _ptr(act), _ptr(y), _ptr(residual), n, width,
-                                   ff, experts, top, _stream()), "moe_grouped", 4)
+                                   ff, experts, top, activation, _ptr(pass_weight), _stream()), "moe_grouped", 4)
 
 
 def moe_grouped_tc_tiles(n_pairs: int, experts: int) -> int:
@@ -1289,11 +1332,12 @@ def moe_grouped_tc_tiles(n_pairs: int, experts: int) -> int:
 def moe_grouped_tc(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
                    weights: torch.Tensor, perm: torch.Tensor, place: torch.Tensor, tile_expert: torch.Tensor,
                    x_sorted: torch.Tensor, act: torch.Tensor, y: torch.Tensor,
-                   residual: torch.Tensor, top: int) -> None:
+                   residual: torch.Tensor, top: int, activation: int = GEMM_ACT_RELU2,
+                   pass_weight: Optional[torch.Tensor] = None) -> None:
     """``moe_grouped`` with both products on the tcgen05 kernel: runs padded to tiles of 128
     rows (``moe_grouped_tc_tiles``), the rows gathered into ``x_sorted`` [tiles * 128, width]
-    first, relu^2 in the first product's epilogue."""
-    _cuda(h, w_up, w_down, ids, weights, perm, place, tile_expert, x_sorted, act, y, residual)
+    first, the activation in the first product's epilogue."""
+    _cuda(h, w_up, w_down, ids, weights, perm, place, tile_expert, x_sorted, act, y, residual, pass_weight)
     n, width = h.shape
     experts, ff, _ = w_up.shape
     rows = moe_grouped_tc_tiles(n * top, experts) * 128
@@ -1309,7 +1353,8 @@ def moe_grouped_tc(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, id
     _need(residual.dtype == torch.float32 and tuple(residual.shape) == (n, width), "moe_grouped_tc: residual")
     _check(_lib().nnis_moe_grouped_tc(_ptr(h), _ptr(w_up), _ptr(w_down), _ptr(ids), _ptr(weights), _ptr(perm),
                                       _ptr(place), _ptr(tile_expert), _ptr(x_sorted), _ptr(act), _ptr(y),
-                                      _ptr(residual), n, width, ff, experts, top, sm_count(h.device),
+                                      _ptr(residual), n, width, ff, experts, top, activation, _ptr(pass_weight),
+                                      sm_count(h.device),
                                       _ptr(status_word(h.device)), PDL, _stream()), "moe_grouped_tc", 5)
 
 
@@ -1544,7 +1589,8 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
              page_table: Optional[torch.Tensor], q_out: torch.Tensor, k_cache: Optional[torch.Tensor],
              v_cache: Optional[torch.Tensor], gate_out: Optional[torch.Tensor], heads: int, kv_heads: int,
              dk: int, dv: int, rot: int, eps: float, pairing: str = "neighbours", head_norm: bool = False,
-             q_scale: Optional[torch.Tensor] = None, maps: int = 1, magnitude: float = 1.0) -> None:
+             q_scale: Optional[torch.Tensor] = None, maps: int = 1, magnitude: float = 1.0,
+             head_weights=None) -> None:
     """From float32 rows [q | k | v | gate logits]: norms of q and k, rotation, q packed, k and v into
     the cache, sigmoid of the gate's logits (``gate_out`` [n, heads] or [n, heads * dv]: as many logits a
     row).  ``kv_heads == 0``: the rows hold no keys and values.  Two forms: with ``wq``/``wk`` the
@@ -1553,7 +1599,12 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
     q) or a gate per value, everything is per head: the rotation (either pairing), then optionally
     every head divided by its own root mean square.  ``maps`` > 1: a head of q or k holds that many
     vectors of dk / maps values side by side, each turned by itself over its first ``rot`` values;
-    ``magnitude`` multiplies every cosine and sine."""
+    ``magnitude`` multiplies every cosine and sine.  ``head_weights``: (q's, k's), float32 [dk] each or
+    None: every head of q (k) normed by itself with that weight, before the rotation (the per-head form)."""
+    hq, hk = head_weights if head_weights is not None else (None, None)
+    _cuda(hq, hk)
+    for w in (hq, hk):
+        _need(w is None or (w.dtype == torch.float32 and w.numel() == dk), "qkv_prep: head_weights float32 [dk]")
     _cuda(a, wq, wk, freq, token_pos, token_seq, page_table, q_out, k_cache, v_cache, gate_out, q_scale)
     n = a.shape[0]
     gate_cols = 0 if gate_out is None else gate_out.shape[1]
@@ -1574,14 +1625,14 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
         _need(page_table is not None and page_table.dtype == torch.int32, "qkv_prep: page_table int32")
         cols, page_size = page_table.shape[1], k_cache.shape[2]
     per_head = head_norm or pairing == "half" or q_scale is not None or gate_cols not in (0, heads) \
-        or maps != 1 or magnitude != 1.0
+        or maps != 1 or magnitude != 1.0 or head_weights is not None
     _need(maps >= 1 and dk % maps == 0 and rot <= dk // maps, "qkv_prep: maps vectors of equal size in a head")
     if per_head:
         _need(wq is None and wk is None, "qkv_prep: the per-head form has no norm over the whole projections")
         _need(q_scale is None or (q_scale.dtype == torch.float32 and q_scale.numel() == heads),
               "qkv_prep: q_scale float32 [heads]")
-        _check(_lib().nnis_qkv_prep_heads(_ptr(a), _ptr(q_scale), _ptr(freq), _ptr(token_pos), _ptr(token_seq),
-                                          _ptr(page_table), cols, _ptr(q_out), _ptr(k_cache), _ptr(v_cache),
+        _check(_lib().nnis_qkv_prep_heads(_ptr(a), _ptr(hq), _ptr(hk), _ptr(q_scale), _ptr(freq), _ptr(token_pos),
+                                          _ptr(token_seq), _ptr(page_table), cols, _ptr(q_out), _ptr(k_cache), _ptr(v_cache),
                                           _ptr(gate_out), n, heads, kv_heads, dk, dv, rot,
                                           1 if pairing == "half" else 0, 1 if head_norm else 0, gate_cols,
                                           page_size, ctypes.c_float(eps), maps, ctypes.c_float(magnitude),
@@ -1598,10 +1649,16 @@ def attention_sink(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor
                    token_seq: torch.Tensor, page_table: torch.Tensor, sink: Optional[torch.Tensor],
                    gate: Optional[torch.Tensor], out: torch.Tensor, heads: int, kv_heads: int, window: int,
                    chunk: int, scale: float, cap: float, n_splits: int = 1,
-                   partial: Optional[torch.Tensor] = None) -> None:
+                   partial: Optional[torch.Tensor] = None, keep: int = 0,
+                   bias: Optional[torch.Tensor] = None) -> None:
     """Causal attention of packed queries over the paged cache with a soft cap on the scores, a
-    chunked and/or windowed mask, a sink per head in the denominator and a gate per (token, head)."""
-    _cuda(q, k_cache, v_cache, token_pos, token_seq, page_table, sink, gate, out, partial)
+    chunked and/or windowed mask, a sink per head in the denominator and a gate per (token, head).
+    ``keep``: the first keys of a sequence that every later query sees whatever the mask says;
+    ``bias`` (float32 [heads, distances]): added to a score by the distance of query and key, the last
+    column for all distances beyond."""
+    _cuda(q, k_cache, v_cache, token_pos, token_seq, page_table, sink, gate, out, partial, bias)
+    _need(bias is None or (bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == heads),
+          "attention_sink: bias float32 [heads, distances]")
     n = out.shape[0]
     pages, nkv, page_size, dk = k_cache.shape
     dv = v_cache.shape[3]
@@ -1620,38 +1677,44 @@ def attention_sink(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor
     _check(_lib().nnis_attention_sink(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(token_pos), _ptr(token_seq),
                                       _ptr(page_table), page_table.shape[1], _ptr(sink), _ptr(gate), _ptr(out),
                                       _ptr(partial), n, heads, kv_heads, dk, dv, page_size, window, chunk,
-                                      ctypes.c_float(scale), ctypes.c_float(cap), n_splits, gate_elems,
+                                      ctypes.c_float(scale), ctypes.c_float(cap), n_splits, gate_elems, keep,
+                                      _ptr(bias), bias.shape[1] if bias is not None else 0,
                                       code_of(out.dtype), _stream()), "attention_sink", 2 if n_splits > 1 else 1)
 
 
 def attention_sink_mma_takes(dk: int, dv: int, page_size: int) -> bool:
     """Whether the tensor-core prompt form of the sink attention takes these head sizes."""
-    return dk == dv and dk in (64, 128) and page_size == 64
+    return bool(_lib().nnis_attention_sink_mma_takes(dk, dv, page_size))
 
 
 def attention_sink_mma(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, tiles: torch.Tensor,
                        seq_first_row: torch.Tensor, seq_start: torch.Tensor, seq_count: torch.Tensor,
                        page_table: torch.Tensor, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor],
                        out: torch.Tensor, heads: int, kv_heads: int, window: int, chunk: int, scale: float,
-                       cap: float) -> None:
+                       cap: float, keep: int = 0, bias: Optional[torch.Tensor] = None) -> None:
     """``attention_sink`` for prompt steps in bfloat16 on mma.sync tiles; ``tiles`` int32 [n, 2] =
     (sequence, first query) per 64 queries."""
-    _cuda(q, k_cache, v_cache, tiles, seq_first_row, seq_start, seq_count, page_table, sink, gate, out)
+    _cuda(q, k_cache, v_cache, tiles, seq_first_row, seq_start, seq_count, page_table, sink, gate, out, bias)
     pages, nkv, page_size, d = k_cache.shape
+    dv = v_cache.shape[3]
     n = out.shape[0]
     _need(q.dtype == k_cache.dtype == v_cache.dtype == out.dtype == torch.bfloat16, "attention_sink_mma: bfloat16")
-    _need(attention_sink_mma_takes(d, v_cache.shape[3], page_size) and nkv == kv_heads,
-          "attention_sink_mma: heads of 64 or 128 for keys and values alike, pages of 64")
-    _need(tuple(q.shape) == tuple(out.shape) == (n, heads * d), "attention_sink_mma: q, out [n, heads * d]")
+    _need(attention_sink_mma_takes(d, dv, page_size) and nkv == kv_heads,
+          "attention_sink_mma: heads of up to 128 values in multiples of eight, pages of 64")
+    _need(tuple(q.shape) == (n, heads * d) and tuple(out.shape) == (n, heads * dv),
+          "attention_sink_mma: q [n, heads * dk], out [n, heads * dv]")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.dim() == 2 and bias.shape[0] == heads),
+          "attention_sink_mma: bias float32 [heads, distances]")
     _need(tiles.dtype == torch.int32 and tiles.dim() == 2 and tiles.shape[1] == 2, "attention_sink_mma: tiles [n, 2]")
     _need(sink is None or (sink.dtype == torch.float32 and sink.numel() == heads), "attention_sink_mma: sink")
     _need(gate is None or (gate.dtype == torch.float32 and gate.numel() >= n * heads), "attention_sink_mma: gate")
-    gate_elems = d if gate is not None and gate.dim() == 2 and gate.shape[1] == heads * d else 0
+    gate_elems = dv if gate is not None and gate.dim() == 2 and gate.shape[1] == heads * dv and dv > 1 else 0
     _check(_lib().nnis_attention_sink_mma(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(tiles), tiles.shape[0],
                                           _ptr(seq_first_row), _ptr(seq_start), _ptr(seq_count), _ptr(page_table),
-                                          page_table.shape[1], _ptr(sink), _ptr(gate), _ptr(out), heads, kv_heads, d,
+                                          page_table.shape[1], _ptr(sink), _ptr(gate), _ptr(out), heads, kv_heads, d, dv,
                                           page_size, window, chunk, ctypes.c_float(scale), ctypes.c_float(cap),
-                                          gate_elems, _stream()), "attention_sink_mma")
+                                          gate_elems, keep, _ptr(bias), bias.shape[1] if bias is not None else 0,
+                                          _stream()), "attention_sink_mma")
 
 
 def moe_experts_gated(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
@@ -1929,10 +1992,14 @@ def attention_diff(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor
 # ---------------------------------------------------------------------------
 def moe_route_choice(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor],
                      token_pos: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, pass_weight: torch.Tensor,
-                     experts: int, top: int, groups: int = 1, keep: int = 1) -> None:
-    """Scores s = softmax over ALL outputs of the router; chosen: the ``top`` largest s + correction among
+                     experts: int, top: int, groups: int = 1, keep: int = 1, sigmoid_scores: bool = False,
+                     group_top: int = 1, renormalise: bool = False) -> None:
+    """Scores s = softmax over ALL outputs of the router (``sigmoid_scores``: the sigmoid of each); chosen: the ``top`` largest s + correction among
     the ``keep`` best of ``groups`` equal runs of neighbours; weights = the chosen s, as they are.  Outputs
-    from ``experts`` on have no expert: ids -1, their weights summed in ``pass_weight`` [n]."""
+    from ``experts`` on have no expert: ids -1, their weights summed in ``pass_weight`` [n].
+    A run's rank is its largest s + correction (``group_top`` 1) or the sum of its two largest (2);
+    ``renormalise``: the weights divided by their sum + 1e-20."""
+    _need(group_top in (1, 2), "moe_route_choice: group_top 1 or 2")
     _cuda(h, w_router, correction, token_pos, ids, weights, pass_weight)
     n, width = h.shape
     outputs = w_router.shape[0]
@@ -1944,7 +2011,8 @@ def moe_route_choice(h: torch.Tensor, w_router: torch.Tensor, correction: Option
           "moe_route_choice: ids int32 [n, top], weights float32 [n, top], pass_weight float32 [n]")
     _check(_lib().nnis_moe_route_choice(_ptr(h), _ptr(w_router), _ptr(correction), _ptr(token_pos), _ptr(ids),
                                         _ptr(weights), _ptr(pass_weight), n, width, outputs, experts, top, groups,
-                                        keep, code_of(h.dtype), _stream()), "moe_route_choice")
+                                        keep, 1 if sigmoid_scores else 0, group_top, 1 if renormalise else 0,
+                                        code_of(h.dtype), _stream()), "moe_route_choice")
 
 
 def moe_experts_gated_out(h: torch.Tensor, w_gu: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,

@@ -236,6 +236,7 @@ class GraphDecoder:
                 table = cache.page_table(g, slot)
                 count = min(len(table), cols)
                 dropped = min(group.first_needed_page(cache.lengths[slot]), count) if group.window > 0 else 0
+                kept = group.kept_pages  # (pages in front of the dropped ones that stay)
                 known = mirror[r]
                 version = cache.versions[slot]
                 same = known is not None and known[0] is table and known[3] == version
@@ -244,7 +245,7 @@ class GraphDecoder:
                 line = st[base + r * cols:base + (r + 1) * cols]
                 if same and known[1] <= count and known[2] <= dropped:
                     line[known[1]:count] = table[known[1]:count]
-                    line[known[2]:dropped] = -1
+                    line[max(known[2], kept):dropped] = -1
                 else:
                     line[:count] = table[:count]
                     line[count:] = -1

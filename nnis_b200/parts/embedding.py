@@ -36,6 +36,17 @@ class TokenEmbedding(Part):
         ops.embed(self.table, tokens, hidden, status)
 
 
+class ScaledTokenEmbedding(TokenEmbedding):
+    """The same times a number, in float32.  params: vocab_size, hidden_size, name, scale."""
+
+    def __init__(self, params, prefix, dtype, device):
+        super().__init__(params, prefix, dtype, device)
+        self.scale = float(params["scale"])
+
+    def forward(self, tokens: torch.Tensor, hidden: torch.Tensor, status: torch.Tensor) -> None:
+        ops.embed(self.table, tokens, hidden, status, self.scale)
+
+
 class NormedTokenEmbedding(TokenEmbedding):
     """The same followed by a norm of the embedded rows (in place, float32).
     params: vocab_size, hidden_size, name, norm (a PartSpec of ``NORMS``)."""
@@ -177,6 +188,7 @@ class LinearHead(Part):
 
 
 EMBEDDINGS.register("token_embedding", TokenEmbedding)
+EMBEDDINGS.register("scaled_token_embedding", ScaledTokenEmbedding)
 EMBEDDINGS.register("normed_token_embedding", NormedTokenEmbedding)
 EMBEDDINGS.register("pair_hash_embedding", PairHashEmbedding)
 HEADS.register("linear_head", LinearHead)

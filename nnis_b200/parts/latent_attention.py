@@ -6,7 +6,13 @@ queries and ``c = rms((W_dkv h)[:kv_rank]) * w_kv`` for keys and values; the las
 rotated by position.  Per head, ``q = W_uq cq`` is ``dim`` plain and ``rot_dim``
 rotated values, the plain key is ``W_uk c`` and the value ``W_uv c``; a score is
 ``(q_plain . k_plain + q_rot . k_rot) * scale`` and the weights an ordinary softmax
-over the positions up to the query's.
+over the positions up to the query's (``window`` > 0: over the last ``window`` of them).
+
+With ``q_rank`` 0 there is no latent for the queries: ``q = W_q h``.  Then the queries, the
+latent and, with ``gate`` "head", the logits of a gate per head (head i's output is multiplied
+by ``sigmoid(W_g h)_i``) come from one product of stacked matrices, and one kernel
+(``latent_prep_direct``) packs, turns, norms, stores and takes the sigmoid; the gate multiplies
+the weighted sum of latents, which is the head's output before its linear ``W_uv``.
 
 Only ``[c | k_rot]`` is cached, one row per position for all heads, in a cache
 group without storage for values.  Because ``q_plain . (W_uk c) = (W_uk^T q_plain) . c``,
@@ -16,9 +22,9 @@ product with the cached row, the output is a weighted sum of the rows' ``c`` par
 and the heads' values are made from that sum (``W_uv`` per head) before ``W_o`` adds
 into the residual stream.  Prompts, later chunks and single tokens take the same way.
 
-params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, eps,
-position (a ``rope_frequencies`` PartSpec), names {dq, dq_norm, uq, dkv, dkv_norm,
-uk, uv, o}.
+params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, eps, window, gate,
+position (a ``rope_frequencies`` PartSpec, either pairing), names {dq, dq_norm, uq (or q), dkv,
+dkv_norm, uk, uv, o, gate}.
 """
 from __future__ import annotations
 
@@ -41,10 +47,17 @@ class LatentAttention(Part):
         self.dim = int(params["dim"])
         self.rot = int(params["rot_dim"])
         self.vdim = int(params["vdim"])
-        self.q_rank = int(params["q_rank"])
+        self.q_rank = int(params.get("q_rank") or 0)  # 0: queries straight from h
         self.kv_rank = int(params["kv_rank"])
         self.scale = float(params["scale"])
         self.eps = float(params["eps"])
+        self.window = int(params.get("window") or 0)
+        gate = params.get("gate", False)
+        if gate not in (False, None, "head"):
+            raise ValueError(f"latent attention: gate {gate!r} is not known (head)")
+        self.has_gate = bool(gate)
+        if self.has_gate and self.q_rank:
+            raise ValueError("latent attention: a gate goes with queries straight from the input (q_rank 0)")
         self.names = params["names"]
         pos = params["position"]
         self.position = POSITIONS.build(pos.kind, pos.params, prefix, dtype, device)
@@ -52,12 +65,14 @@ class LatentAttention(Part):
             raise ValueError("latent attention rotates by a table of frequencies (rope_frequencies)")
         if self.position.dims > self.rot:
             raise ValueError(f"rotation over {self.position.dims} dimensions, the rotated part has {self.rot}")
-        for what in ("heads", "dim", "vdim", "q_rank", "kv_rank"):
+        self.pairing = getattr(self.position, "pairing", "half")
+        for what in ("heads", "dim", "vdim", "kv_rank"):
             if getattr(self, what) <= 0:
                 raise ValueError(f"latent attention: {what} must be positive")
         if self.kv_rank > 512:
             raise ValueError("latent attention kernels take latents of up to 512 values")
         self.row = self.kv_rank + self.rot  # a cached row, and a query in the latent's space
+        self.q_cols = self.heads * (self.dim + self.rot)
         self.w_down = self.w_uq = self.w_ukt = self.w_uv = self.w_o = None
         self.norm_q = self.norm_kv = None
 
@@ -67,24 +82,37 @@ class LatentAttention(Part):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         W, H = self.hidden, self.heads
-        return {
-            self._name("dq"): WeightSpec((self.q_rank, W), "matrix", fan_in=W),
-            self._name("dq_norm"): WeightSpec((self.q_rank,), "vector", init="ones"),
-            self._name("uq"): WeightSpec((H * (self.dim + self.rot), self.q_rank), "matrix", fan_in=self.q_rank),
+        if self.q_rank:
+            specs = {
+                self._name("dq"): WeightSpec((self.q_rank, W), "matrix", fan_in=W),
+                self._name("dq_norm"): WeightSpec((self.q_rank,), "vector", init="ones"),
+                self._name("uq"): WeightSpec((self.q_cols, self.q_rank), "matrix", fan_in=self.q_rank),
+            }
+        else:
+            specs = {self._name("q"): WeightSpec((self.q_cols, W), "matrix", fan_in=W)}
+        if self.has_gate:
+            specs[self._name("gate")] = WeightSpec((H, W), "matrix", fan_in=W)
+        specs.update({
             self._name("dkv"): WeightSpec((self.kv_rank + self.rot, W), "matrix", fan_in=W),
             self._name("dkv_norm"): WeightSpec((self.kv_rank,), "vector", init="ones"),
             self._name("uk"): WeightSpec((H * self.dim, self.kv_rank), "matrix", fan_in=self.kv_rank),
             self._name("uv"): WeightSpec((H * self.vdim, self.kv_rank), "matrix", fan_in=self.kv_rank),
             self._name("o"): WeightSpec((W, H * self.vdim), "matrix", fan_in=H * self.vdim),
-        }
+        })
+        return specs
 
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         H = self.heads
-        # both down-projections read h: one product [q latent | c raw | k_rot raw]
-        self.w_down = torch.cat([tensors[self._name("dq")], tensors[self._name("dkv")]], 0).contiguous()
-        self.norm_q = tensors[self._name("dq_norm")]
+        # what reads h is one product: [q latent | c raw | k_rot raw], or [q | c raw | k_rot raw | gate]
+        keys = ["dq" if self.q_rank else "q", "dkv"] + (["gate"] if self.has_gate else [])
+        rows = [tensors[self._name(k)] for k in keys]
+        if not self.q_rank:  # zero rows up to a multiple of eight, as the decode projection kernels take them
+            rows.append(rows[0].new_zeros((-sum(r.shape[0] for r in rows) % 8, self.hidden)))
+        self.w_down = torch.cat(rows, 0).contiguous()
+        if self.q_rank:
+            self.norm_q = tensors[self._name("dq_norm")]
+            self.w_uq = tensors[self._name("uq")]
         self.norm_kv = tensors[self._name("dkv_norm")]
-        self.w_uq = tensors[self._name("uq")]
         # per head [kv_rank, dim]: the product that carries q_plain into the latent's space
         self.w_ukt = tensors[self._name("uk")].view(H, self.dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = tensors[self._name("uv")].view(H, self.vdim, self.kv_rank).contiguous()
@@ -92,11 +120,12 @@ class LatentAttention(Part):
 
     def parameter_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in
-                   (self.w_down, self.w_uq, self.w_ukt, self.w_uv, self.w_o, self.norm_q, self.norm_kv))
+                   (self.w_down, self.w_uq, self.w_ukt, self.w_uv, self.w_o, self.norm_q, self.norm_kv)
+                   if t is not None)
 
     # -- cache ------------------------------------------------------------
     def cache_request(self) -> Optional[KVRequest]:
-        return KVRequest(1, self.row, 0, values=False)
+        return KVRequest(1, self.row, self.window, values=False)
 
     def check_shared_cache(self, view: KVView) -> None:
         raise ValueError("latent attention writes a cache of its own")
@@ -104,9 +133,10 @@ class LatentAttention(Part):
     def step_flops(self, counts, starts) -> float:
         H, W = self.heads, self.hidden
         tokens = sum(counts)
-        per_token = W * (self.q_rank + self.row) + self.q_rank * H * (self.dim + self.rot) \
-            + H * self.dim * self.kv_rank + H * self.vdim * self.kv_rank + H * self.vdim * W
-        keys = sum(c * st + c * (c + 1) // 2 for c, st in zip(counts, starts))
+        into_q = W * self.q_rank + self.q_rank * self.q_cols if self.q_rank else W * (self.q_cols + (H if self.has_gate else 0))
+        per_token = into_q + W * self.row + H * self.dim * self.kv_rank + H * self.vdim * self.kv_rank + H * self.vdim * W
+        keys = sum(sum(min(st + q + 1, self.window) for q in range(c)) if self.window
+                   else c * st + c * (c + 1) // 2 for c, st in zip(counts, starts))
         return 2.0 * tokens * per_token + 2.0 * H * (self.row + self.kv_rank) * keys
 
     # -- work lists ---------------------------------------------------------
@@ -128,7 +158,8 @@ class LatentAttention(Part):
         """Slices of the key range in a step of single tokens: enough CTAs for two per SM,
         at least two pages a slice."""
         ctas = n * -(-self.heads // ops.latent_tile_rows(self.kv_rank)) * -(-self.kv_rank // 512)
-        pages = max(1, -(-ctx.max_context // PAGE_SIZE))
+        keys = ctx.max_context if not self.window else min(ctx.max_context, self.window + PAGE_SIZE - 1)
+        pages = max(1, -(-keys // PAGE_SIZE))
         want = -(-2 * ops.sm_count(self.device) // max(1, ctas * max(1, ctx.share)))
         return int(max(1, min(want, pages // 2, 64)))
 
@@ -138,18 +169,18 @@ class LatentAttention(Part):
         H, ws = self.heads, ctx.workspace
         table = ctx.page_tables[cache.group]
         freq = self.position.frequencies()
-        down = ws.get("latent_down", (n, self.q_rank + self.row), torch.float32)
+        down = ws.get("latent_down", (n, self.w_down.shape[0]), torch.float32)
         linear(x, self.w_down, None, down, STORE_F32, decode=ctx.decode)
-        cq = ws.get("latent_cq", (n, self.q_rank), self.dtype)
-        ops.latent_prep(down, self.norm_q, self.norm_kv, freq, ctx.token_pos, ctx.token_seq, table, cq,
-                        cache.k, self.q_rank, self.kv_rank, self.rot, self.position.dims, self.eps)
-        q = ws.get("latent_q", (n, H * (self.dim + self.rot)), self.dtype)
-        linear(cq, self.w_uq, None, q, STORE, decode=ctx.decode)
         q_lat = ws.get("latent_q_abs", (n, H * self.row), self.dtype)
-        ops.batched_linear(q, self.dim + self.rot, self.w_ukt, q_lat, self.row)
-        if self.rot:
-            ops.rope_part(q, self.dim + self.rot, self.dim, q_lat, self.row, self.kv_rank, ctx.token_pos,
-                          freq, H, self.rot, self.position.dims)
+        gate = ws.get("latent_gate", (n, H), torch.float32) if self.has_gate else None
+        if self.q_rank:
+            self._queries_from_latent(ctx, down, q_lat, freq, table, cache)
+        else:
+            q = ws.get("latent_q", (n, H * self.dim), self.dtype)
+            ops.latent_prep_direct(down, self.norm_kv, freq, ctx.token_pos, ctx.token_seq, table, q, q_lat, cache.k,
+                                   gate, H, self.dim, self.kv_rank, self.rot, self.position.dims, self.eps,
+                                   pairing=self.pairing)
+            ops.batched_linear(q, self.dim, self.w_ukt, q_lat, self.row)
         o_lat = ws.get("latent_o", (n, H * self.kv_rank), self.dtype)
         tiles = ctx.tables.get(self._tiles_name())
         if self._tensor_cores() and (ctx.decode or tiles is not None):
@@ -158,20 +189,37 @@ class LatentAttention(Part):
                 if splits > 1 else None
             if ctx.decode:
                 ops.attention_latent_mma(q_lat, cache.k, None, None, None, None, ctx.token_pos, ctx.token_seq,
-                                         table, o_lat, H, self.kv_rank, self.scale, splits, partial)
+                                         table, o_lat, H, self.kv_rank, self.scale, splits, partial,
+                                         window=self.window, gate=gate)
             else:
                 ops.attention_latent_mma(q_lat, cache.k, tiles, ctx.seq_first_row, ctx.seq_start,
                                          ctx.seq_count, ctx.token_pos, ctx.token_seq, table, o_lat, H,
-                                         self.kv_rank, self.scale)
+                                         self.kv_rank, self.scale, window=self.window, gate=gate)
         else:
             splits = ctx.attention_splits(n * H)
+            if self.window:  # a slice has at least 64 keys of the window
+                splits = max(1, min(splits, -(-self.window // 64)))
             partial = ws.get("attn_partial", (n * H * splits * (self.kv_rank + 2),), torch.float32) \
                 if splits > 1 else None
             ops.attention_latent(q_lat, cache.k, ctx.token_pos, ctx.token_seq, table, o_lat, H, self.kv_rank,
-                                 self.scale, splits, partial)
+                                 self.scale, splits, partial, window=self.window, gate=gate)
         attn = ws.get("attn", (n, H * self.vdim), self.dtype)
         ops.batched_linear(o_lat, self.kv_rank, self.w_uv, attn, self.vdim)
         linear(attn, self.w_o, None, residual, ADD_F32, ws, decode=ctx.decode)
+
+    def _queries_from_latent(self, ctx, down, q_lat, freq, table, cache) -> None:
+        """Queries by way of their own latent: norm, up-projection, into the latent's space."""
+        n, H, ws = down.shape[0], self.heads, ctx.workspace
+        cq = ws.get("latent_cq", (n, self.q_rank), self.dtype)
+        ops.latent_prep(down, self.norm_q, self.norm_kv, freq, ctx.token_pos, ctx.token_seq, table, cq,
+                        cache.k, self.q_rank, self.kv_rank, self.rot, self.position.dims, self.eps,
+                        pairing=self.pairing)
+        q = ws.get("latent_q", (n, self.q_cols), self.dtype)
+        linear(cq, self.w_uq, None, q, STORE, decode=ctx.decode)
+        ops.batched_linear(q, self.dim + self.rot, self.w_ukt, q_lat, self.row)
+        if self.rot:
+            ops.rope_part(q, self.dim + self.rot, self.dim, q_lat, self.row, self.kv_rank, ctx.token_pos,
+                          freq, H, self.rot, self.position.dims, pairing=self.pairing)
 
 
 MIXERS.register("latent_attention", LatentAttention)

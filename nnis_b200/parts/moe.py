@@ -1,7 +1,7 @@
 """Mixture of experts: every token runs ``top`` of ``experts`` small feed-forward
 layers and, optionally, a shared one.
 
-An expert is ``W_down act(W_up h)`` with act = relu squared, no biases.  The router's
+An expert is ``W_down act(W_up h)`` with act = relu squared or the erf gelu, no biases.  The router's
 logits ``z = W_r h + b`` are float32 (its matrix is kept in float32); the ``top``
 largest choose the experts and a softmax over the chosen logits alone weighs them.
 The shared expert has the same form, runs for every token and is multiplied by
@@ -25,18 +25,21 @@ Prompt steps in bfloat16 sort the pairs by expert and run grouped products: on m
 (score and activation in the first product's epilogue) where an expert gets few rows, on the
 tcgen05 kernel (float32 sums, then a row-wise kernel for score and activation) where it gets many.
 
-A third form (``scores`` "softmax_all" with gated experts and ``weight_on`` "output"): the scores
-are ONE softmax over all the router's outputs; the choice goes by score + a stored correction per
+A third form (``scores`` "softmax_all" with ``weight_on`` "output"): the scores
+are ONE softmax over all the router's outputs (``scores`` "sigmoid_all": the sigmoid of each output's
+logit); the choice goes by score + a stored correction per
 output (``names["correction"]``), group by group (``groups`` equal runs of neighbouring outputs, a
-run's score its largest corrected score, only the ``keep`` best runs can be chosen), and the chosen
-scores weigh the experts' OUTPUTS as they are, not renormalised.  The router's last ``identity``
+run's score its largest corrected score, or with ``group_top`` 2 the sum of its two largest, only the
+``keep`` best runs can be chosen), and the chosen scores weigh the experts' OUTPUTS as they are
+(``renormalise``: divided by their sum + 1e-20).  Experts are gated or plain ("relu2", "gelu").  The router's last ``identity``
 outputs have no matrices: such an expert hands its input on, so the token's output takes weight *
 h from it.  The shared expert of this form is a gated feed-forward of its own (``shared``: a
 ``gated_mlp`` PartSpec) that runs for every token.
 
 params: hidden_size, experts, top, ff, shared_ff (0: no shared expert), activation
-("relu2" | "silu_gated"), scores ("softmax" over the chosen logits | "sigmoid" | "softmax_all"),
-weight_on ("output" | "input"), identity, groups, keep, shared (a PartSpec), names {router,
+("relu2" | "gelu", with erf | "silu_gated"), scores ("softmax" over the chosen logits | "sigmoid" |
+"softmax_all" | "sigmoid_all"), weight_on ("output" | "input"), identity, groups, keep, group_top,
+renormalise, shared (a PartSpec), names {router,
 router_bias (optional), correction (optional), expert (a format with {e}), up, down, gate (gated
 experts), shared_up, shared_down, shared_gate}.
 """
@@ -55,6 +58,7 @@ from .linear import ADD_F32, STORE_F32, linear
 
 class MoEFeedForward(Part):
     GROUPED_FROM = 32  # tokens of a prompt step from which the pairs are sorted by expert
+    PLAIN_ACTIVATIONS = {"relu2": ops.GEMM_ACT_RELU2, "gelu": ops.GEMM_ACT_GELU_ERF}
     TCGEN05_ROWS = 96  # (token, expert) pairs an expert on average from which runs are padded to 128 rows
 
     def __init__(self, params, prefix, dtype, device):
@@ -71,18 +75,27 @@ class MoEFeedForward(Part):
         self.identity = int(params.get("identity") or 0)
         self.groups = int(params.get("groups") or 1)
         self.keep = int(params.get("keep") or self.groups)
-        self.by_choice = self.scores == "softmax_all"
-        if (self.activation, self.scores, self.weight_on) not in (("relu2", "softmax", "output"),
-                                                                  ("silu_gated", "sigmoid", "input"),
-                                                                  ("silu_gated", "softmax_all", "output")):
+        self.group_top = int(params.get("group_top") or 1)
+        self.renormalise = bool(params.get("renormalise", False))
+        self.by_choice = self.scores in ("softmax_all", "sigmoid_all")
+        plain = self.activation in self.PLAIN_ACTIVATIONS
+        known = (plain and self.scores == "softmax" and self.weight_on == "output") \
+            or (self.activation == "silu_gated" and self.scores == "sigmoid" and self.weight_on == "input") \
+            or ((plain or self.activation == "silu_gated") and self.by_choice and self.weight_on == "output")
+        if not known:
             raise ValueError(f"moe: no kernel for activation {self.activation!r} with {self.scores!r} scores "
                              f"on the expert's {self.weight_on}")
         self.gated = self.activation == "silu_gated"
-        if self.gated and self.shared_ff:
-            raise ValueError("moe: the gated form's shared expert is a part of its own (shared)")
+        self.act = self.PLAIN_ACTIVATIONS.get(self.activation)
+        if (self.gated or self.by_choice) and self.shared_ff:
+            raise ValueError("moe: this form's shared expert is a part of its own (shared)")
         self.outputs = self.experts + self.identity  # of the router
-        if not self.by_choice and (self.identity or self.groups != 1 or params.get("shared") is not None):
-            raise ValueError("moe: identity experts, groups and a shared part go with softmax_all scores")
+        if not self.by_choice and (self.identity or self.groups != 1 or params.get("shared") is not None
+                                   or self.group_top != 1 or self.renormalise):
+            raise ValueError("moe: identity experts, groups, renormalised weights and a shared part go with "
+                             "softmax_all or sigmoid_all scores")
+        if self.group_top not in (1, 2):
+            raise ValueError(f"moe: a group is ranked by its largest score or its two largest; got {self.group_top}")
         if not 0 < self.top <= self.outputs:
             raise ValueError(f"moe: top={self.top} of {self.outputs} experts")
         if self.groups <= 0 or self.outputs % self.groups or not 0 < self.keep <= self.groups \
@@ -205,6 +218,17 @@ class MoEFeedForward(Part):
             act = ws.get("moe_act", (n, self.top, self.ff), self.dtype)
             ops.moe_experts_gated(x, self.w_up, self.w_down, ids, weights, ctx.token_pos, act, residual, self.top)
             return
+        self._plain_experts(x, ctx, residual, ids, weights, None)
+        if self.shared_ff:
+            up = ws.get("moe_shared_up", (n, self.w_shared_up.shape[0]), torch.float32)
+            linear(x, self.w_shared_up, None, up, STORE_F32, decode=ctx.decode)
+            shared_act = ws.get("moe_shared_act", (n, self.shared_ff), self.dtype)
+            ops.relu2_gate(up, shared_act)
+            linear(shared_act, self.w_shared_down, None, residual, ADD_F32, ws, decode=ctx.decode)
+
+    def _plain_experts(self, x, ctx, residual, ids, weights, pass_weight) -> None:
+        """The chosen experts W_down act(W_up x), their outputs weighted; ``pass_weight``: see the module's text."""
+        n, ws = residual.shape[0], ctx.workspace
         grouped = self.dtype == torch.bfloat16 and not ctx.decode and n >= self.GROUPED_FROM \
             and ops.moe_grouped_takes(self.hidden, self.ff, self.experts)
         if grouped and ops.TC_GEMM and n * self.top >= self.TCGEN05_ROWS * self.experts:
@@ -217,7 +241,7 @@ class MoEFeedForward(Part):
                                ws.get("moe_x_sorted", (tiles * 128, self.hidden), self.dtype),
                                ws.get("moe_act_sorted", (tiles * 128, self.ff), self.dtype),
                                ws.get("moe_y_sorted", (tiles * 128, self.hidden), torch.float32), residual,
-                               self.top)
+                               self.top, self.act, pass_weight)
         elif grouped:
             # pairs sorted by expert in runs padded to 64 rows, grouped products on mma.sync tiles
             tiles = ops.moe_grouped_tiles(n * self.top, self.experts)
@@ -226,26 +250,27 @@ class MoEFeedForward(Part):
                             ws.get("moe_place", (n * self.top,), torch.int32),
                             ws.get("moe_tile_expert", (tiles,), torch.int32),
                             ws.get("moe_act_sorted", (tiles * 64, self.ff), self.dtype),
-                            ws.get("moe_y_sorted", (tiles * 64, self.hidden), torch.float32), residual, self.top)
+                            ws.get("moe_y_sorted", (tiles * 64, self.hidden), torch.float32), residual, self.top, self.act,
+                            pass_weight)
         else:
             act = ws.get("moe_act", (n, self.top, self.ff), self.dtype)
-            ops.moe_experts(x, self.w_up, self.w_down, ids, weights, ctx.token_pos, act, residual, self.top)
-        if self.shared_ff:
-            up = ws.get("moe_shared_up", (n, self.w_shared_up.shape[0]), torch.float32)
-            linear(x, self.w_shared_up, None, up, STORE_F32, decode=ctx.decode)
-            shared_act = ws.get("moe_shared_act", (n, self.shared_ff), self.dtype)
-            ops.relu2_gate(up, shared_act)
-            linear(shared_act, self.w_shared_down, None, residual, ADD_F32, ws, decode=ctx.decode)
-
+            ops.moe_experts(x, self.w_up, self.w_down, ids, weights, ctx.token_pos, act, residual, self.top, self.act,
+                            pass_weight)
 
     def _forward_by_choice(self, x, ctx, residual, ids, weights) -> None:
-        """The form whose scores are one softmax over all outputs (see the module's text)."""
+        """The forms that score all outputs and choose by corrected scores (see the module's text)."""
         n = residual.shape[0]
         ws = ctx.workspace
         passed = ws.get("moe_pass_weight", (n,), torch.float32)
         ops.moe_route_choice(x, self.w_router, self.correction, ctx.token_pos, ids, weights, passed, self.experts,
-                             self.top, self.groups, self.keep)
+                             self.top, self.groups, self.keep, sigmoid_scores=self.scores == "sigmoid_all",
+                             group_top=self.group_top, renormalise=self.renormalise)
         pass_weight = passed if self.identity else None
+        if not self.gated:
+            self._plain_experts(x, ctx, residual, ids, weights, pass_weight)
+            if self.shared is not None:
+                self.shared.forward(x, ctx, residual)
+            return
         grouped = self.dtype == torch.bfloat16 and not ctx.decode and n >= self.GROUPED_FROM and ops.MOE_GROUPED \
             and ops.moe_grouped_takes(self.hidden, self.ff, self.experts)
         if grouped and ops.TC_GEMM and n * self.top >= self.TCGEN05_ROWS * self.experts:

@@ -7,15 +7,24 @@ i reads key/value head i // (H / G)) with values of ``vdim``:
 * q = W_q h, k = W_k h, v = W_v h, no biases.  With ``qk_norm`` (True) q and k are divided by
   their root mean square taken over the WHOLE projection (all heads at once) and
   multiplied by a weight per column, before the rotation.  With ``qk_norm == "head"`` every
-  head of q and of k is divided by its own root mean square AFTER the rotation, without a weight.
-* q and k are rotated by position over the first ``dims`` values of every head (the
+  head of q and of k is divided by its own root mean square AFTER the rotation, without a weight;
+  with ``qk_norm == "head_weight"`` by its own root mean square BEFORE the rotation and multiplied by
+  a weight per value of a head, which all heads share.
+* q and k are rotated by position (``dims`` 0: not at all) over the first ``dims`` values of every head (the
   position encoding's frequencies; neighbouring pairs, or, for an encoding whose ``pairing`` is
   "half", value i with value i + dims / 2).
 * With ``head_scale`` the scores of head i are also multiplied by a learned number per head
   (names["head_scale"]: a temperature); it is folded into q.
 * score = cap * tanh(scale * q.k / cap) (``softcap`` 0: no cap); a query at position p sees
   keys j <= p of its own chunk (``chunk`` > 0: floor(j / chunk) == floor(p / chunk), chunks
-  counted from position 0 of the sequence) and window (``window`` > 0: j > p - window).
+  counted from position 0 of the sequence) and window (``window`` > 0: j > p - window), and
+  whatever the two say the sequence's first ``keep_first`` keys.
+* With ``distance_bias`` {"far": D, "rows": of a table made at random} a score gains, after scale and cap, a learned number by the
+  distance n = p - j and the head: row ``bucket(n)`` of a table of B rows (names["distance_bias"]; B
+  is the stored tensor's).  With h = B // 2 the first h distances have a bucket each, the others share
+  the rest logarithmically up to D: min(B - 1, h + floor(ln(n / h) / ln(D / h) * (B - h))).  At load the
+  table is laid out by distance, up to the first distance of the last bucket, which stands for all
+  beyond it.
 * With ``sink`` the softmax's denominator also holds exp(sink_i), a learned number per
   head with no key and no value.
 * With ``gate`` (True or "head") head i's output is multiplied by sigmoid(W_g h)_i before W_o; with
@@ -27,15 +36,17 @@ part has no k/v projection, norm or cache of its own and reads another schedule 
 One projection makes q, k, v and the gate's logits in float32 (their matrices are
 stacked at load); ``qkv_prep`` norms, rotates, stores and takes the sigmoid; the attention
 kernel serves prompts, later portions and single tokens alike; prompt steps in bfloat16 with
-key and value heads of 64 or 128 run a tensor-core form of it (``attention_sink_mma``).
+key and value heads of up to 128 values (multiples of eight) run a tensor-core form of it
+(``attention_sink_mma``).
 
-params: hidden_size, heads, kv_heads, dim, vdim, scale, softcap, chunk, window, sink,
-gate, qk_norm, head_scale, eps, position (a ``rope_frequencies`` PartSpec),
-kv ("own" | "shared"), names {q, k, v, o, q_norm, k_norm, sink, gate, head_scale}.
+params: hidden_size, heads, kv_heads, dim, vdim, scale, softcap, chunk, window, keep_first,
+distance_bias, sink, gate, qk_norm, head_scale, eps, position (a ``rope_frequencies`` PartSpec),
+kv ("own" | "shared"), names {q, k, v, o, q_norm, k_norm, sink, gate, head_scale, distance_bias}.
 """
 from __future__ import annotations
 
-from typing import Dict, Mapping, Optional
+from fractions import Fraction
+from typing import Dict, List, Mapping, Optional
 
 import numpy as np
 import torch
@@ -45,6 +56,33 @@ from ..csrc import ops
 from ..weights.loader import WeightSpec
 from .base import MIXERS, POSITIONS, Part
 from .linear import ADD_F32, STORE_F32, linear
+
+
+def distance_buckets(buckets: int, far) -> List[int]:
+    """The bucket of every distance 0, 1, ... up to the first distance of the last bucket (all distances
+    beyond are in it too).  Bucket h + k begins at h * (far / h)^(k / m), m = buckets - h; the borders are
+    compared as (n / h)^m against (far / h)^k in exact arithmetic, so that a border that is a whole
+    number belongs to the bucket it opens."""
+    h = buckets // 2
+    m = buckets - h
+    if buckets < 2 or not far > h:
+        raise ValueError(f"distance bias: {buckets} rows up to distance {far}: wants at least two rows and a "
+                         f"distance beyond half of them")
+    ratio = Fraction(far) / h
+    # first distance of every later bucket: the least n with (n / h)^m >= ratio^k
+    first = []
+    for k in range(m):
+        want = ratio ** k
+        n = max(h, int(h * float(ratio) ** (k / m)) - 2)
+        while Fraction(n, h) ** m < want:
+            n += 1
+        first.append(n)
+    out, b = list(range(h)), 0
+    for n in range(h, first[-1] + 1):
+        while b + 1 < m and first[b + 1] <= n:
+            b += 1
+        out.append(h + b)
+    return out
 
 
 class SinkAttention(Part):
@@ -59,6 +97,11 @@ class SinkAttention(Part):
         self.softcap = float(params.get("softcap") or 0.0)
         self.chunk = int(params.get("chunk") or 0)
         self.window = int(params.get("window") or 0)
+        self.keep_first = int(params.get("keep_first") or 0) if (self.chunk or self.window) else 0
+        bias = params.get("distance_bias")
+        self.bias_far = bias["far"] if bias else None
+        self.bias_rows = int(bias.get("rows") or 0) if bias else 0  # of a table made at random
+        self.bias = None  # float32 [heads, distances]
         self.has_sink = bool(params.get("sink", False))
         gate = params.get("gate", False)
         if gate not in (False, True, None, "head", "value"):
@@ -66,24 +109,27 @@ class SinkAttention(Part):
         self.has_gate = bool(gate)
         self.gate_by_value = gate == "value"
         norm = params.get("qk_norm", False)
-        if norm not in (False, True, None, "whole", "head"):
-            raise ValueError(f"sink attention: qk_norm {norm!r} is not known (whole, head)")
+        if norm not in (False, True, None, "whole", "head", "head_weight"):
+            raise ValueError(f"sink attention: qk_norm {norm!r} is not known (whole, head, head_weight)")
         self.head_norm = norm == "head"
-        self.qk_norm = bool(norm) and not self.head_norm
+        self.head_weight_norm = norm == "head_weight"
+        self.qk_norm = bool(norm) and not self.head_norm and not self.head_weight_norm
         self.has_head_scale = bool(params.get("head_scale", False))
         self.eps = float(params.get("eps", 1e-6))
         self.own_kv = params.get("kv", "own") == "own"
         self.names = params["names"]
         if self.heads % self.kv_heads:
             raise ValueError(f"heads={self.heads} is not a multiple of kv_heads={self.kv_heads}")
-        if self.dim % 2 or not 0 < self.dim <= 1024 or not 0 < self.vdim <= 256:
-            raise ValueError(f"sink attention takes even key sizes up to 1024 and value sizes up to 256; "
+        if not 0 < self.dim <= 1024 or not 0 < self.vdim <= 256:
+            raise ValueError(f"sink attention takes key sizes up to 1024 and value sizes up to 256; "
                              f"got {self.dim}, {self.vdim}")
         pos = params["position"]
         self.position = POSITIONS.build(pos.kind, pos.params, prefix, dtype, device)
         if not hasattr(self.position, "frequencies"):
             raise ValueError("sink attention rotates by a table of frequencies")
         self.pairing = getattr(self.position, "pairing", "neighbours")
+        if self.dim % 2 and (self.qk_norm or self.pairing == "neighbours") and not self.head_weight_norm:
+            raise ValueError(f"sink attention: neighbouring pairs want an even key size; got {self.dim}")
         if self.qk_norm and self.pairing != "neighbours":
             raise ValueError("sink attention: the norm over whole projections goes with neighbouring pairs")
         if self.position.dims > self.dim:
@@ -111,6 +157,12 @@ class SinkAttention(Part):
             specs[self._name("q_norm")] = WeightSpec((self.heads * self.dim,), "vector", init="ones")
             if self.own_kv:
                 specs[self._name("k_norm")] = WeightSpec((self.kv_heads * self.dim,), "vector", init="ones")
+        if self.head_weight_norm:
+            specs[self._name("q_norm")] = WeightSpec((self.dim,), "vector", init="ones")
+            if self.own_kv:
+                specs[self._name("k_norm")] = WeightSpec((self.dim,), "vector", init="ones")
+        if self.bias_far is not None:
+            specs[self._name("distance_bias")] = WeightSpec((-1, self.heads), "vector", free=self.bias_rows)
         if self.has_sink:
             specs[self._name("sink")] = WeightSpec((self.heads,), "vector")
         if self.has_head_scale:
@@ -120,9 +172,13 @@ class SinkAttention(Part):
     def load(self, tensors: Mapping[str, torch.Tensor]) -> None:
         self.w_in = torch.cat([tensors[self._name(p)] for p, _ in self._projections()], 0).contiguous()
         self.w_o = tensors[self._name("o")]
-        if self.qk_norm:
+        if self.qk_norm or self.head_weight_norm:
             self.q_norm = tensors[self._name("q_norm")]
             self.k_norm = tensors[self._name("k_norm")] if self.own_kv else None
+        if self.bias_far is not None:
+            table = tensors[self._name("distance_bias")]
+            rows = torch.tensor(distance_buckets(table.shape[0], self.bias_far), device=table.device)
+            self.bias = table[rows].t().contiguous()
         if self.has_sink:
             self.sink = tensors[self._name("sink")]
         if self.has_head_scale:
@@ -134,12 +190,14 @@ class SinkAttention(Part):
     # -- cache ------------------------------------------------------------
     def cache_request(self) -> Optional[KVRequest]:
         # (a chunked mask frees no pages: a layer that shares this cache may have another mask)
-        return KVRequest(self.kv_heads, self.dim, self.window, True, self.vdim) if self.own_kv else None
+        return KVRequest(self.kv_heads, self.dim, self.window, True, self.vdim, self.keep_first if self.window else 0) \
+            if self.own_kv else None
 
     def check_shared_cache(self, view: KVView) -> None:
         if not isinstance(view, KVView) or view.v is None \
                 or tuple(view.k.shape[1:]) != (self.kv_heads, view.page_size, self.dim) \
-                or view.v.shape[3] != self.vdim or (view.window and view.window != self.window):
+                or view.v.shape[3] != self.vdim \
+                or (view.window and (view.window, view.keep_first) != (self.window, self.keep_first)):
             raise ValueError("the shared cache does not fit this attention's heads, sizes or window")
 
     def step_flops(self, counts, starts) -> float:
@@ -152,7 +210,7 @@ class SinkAttention(Part):
                 lo = max(0, p - self.window + 1) if self.window else 0
                 if self.chunk:
                     lo = max(lo, p // self.chunk * self.chunk)
-                keys += p + 1 - lo
+                keys += p + 1 - lo + min(self.keep_first, lo)
             flops += 2.0 * H * (self.dim + self.vdim) * keys
         return flops
 
@@ -178,21 +236,27 @@ class SinkAttention(Part):
         linear(x, self.w_in, None, rows, STORE_F32, decode=ctx.decode)
         q = ws.get("sink_attention_q", (n, H * self.dim), self.dtype)
         gate = ws.get("sink_attention_gate", (n, self.gate_cols), torch.float32) if self.has_gate else None
-        ops.qkv_prep(rows, self.q_norm, self.k_norm, self.position.frequencies(), ctx.token_pos, ctx.token_seq,
+        whole = not self.head_weight_norm
+        ops.qkv_prep(rows, self.q_norm if whole else None, self.k_norm if whole else None,
+                     self.position.frequencies(), ctx.token_pos, ctx.token_seq,
                      table if G else None, q, cache.k if G else None, cache.v if G else None, gate, H, G,
                      self.dim, self.vdim, self.position.dims, self.eps, pairing=self.pairing,
-                     head_norm=self.head_norm, q_scale=self.head_scale)
+                     head_norm=self.head_norm, q_scale=self.head_scale,
+                     head_weights=None if whole else (self.q_norm, self.k_norm))
         out = ws.get("sink_attention_out", (n, H * self.vdim), self.dtype)
         if not ctx.decode and self._mma_prompt() and self.TILES_64 in ctx.tables:
             ops.attention_sink_mma(q, cache.k, cache.v, ctx.tables[self.TILES_64], ctx.seq_first_row, ctx.seq_start,
                                    ctx.seq_count, table, self.sink, gate, out, H, self.kv_heads, self.window,
-                                   self.chunk, self.scale, self.softcap)
+                                   self.chunk, self.scale, self.softcap, self.keep_first, self.bias)
             linear(out, self.w_o, None, residual, ADD_F32, ws, decode=ctx.decode)
             return
         splits = ctx.attention_splits(n * H)
+        if self.window and not self.chunk:  # a slice has at least 64 keys of the window
+            splits = max(1, min(splits, -(-(self.window + self.keep_first) // 64)))
         partial = ws.get("attn_partial", (n * H * splits * (self.vdim + 2),), torch.float32) if splits > 1 else None
         ops.attention_sink(q, cache.k, cache.v, ctx.token_pos, ctx.token_seq, table, self.sink, gate, out, H,
-                           self.kv_heads, self.window, self.chunk, self.scale, self.softcap, splits, partial)
+                           self.kv_heads, self.window, self.chunk, self.scale, self.softcap, splits, partial,
+                           self.keep_first, self.bias)
         linear(out, self.w_o, None, residual, ADD_F32, ws, decode=ctx.decode)
 
 

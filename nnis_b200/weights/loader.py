@@ -43,6 +43,7 @@ class WeightSpec:
     role: str  # "matrix" | "vector" | "table" (integer) | "unused" (may be stored; never read, never missed)
     init: str = "normal"  # random mode: "normal" around 0, "ones" around 1
     fan_in: int = 0  # random mode: inputs summed per output (0: not a projection)
+    free: int = 0  # random mode: what an extent of -1 is made with (0: refused)
 
 
 def shape_fits(shape, wanted) -> bool:

@@ -49,10 +49,11 @@ def random_tensors(wanted: Mapping[str, WeightSpec], seed: int, std: float = 0.0
         gen.manual_seed(tensor_seed(seed, name))
         if spec.role == "unused":
             continue
-        if any(extent < 0 for extent in spec.shape):
+        shape = tuple(spec.free if extent < 0 else extent for extent in spec.shape)
+        if any(extent <= 0 for extent in shape):
             raise ValueError(f"{name}: the configuration leaves an extent of {list(spec.shape)} to the stored "
                              f"tensor; random weights need it named")
-        x = torch.randn(spec.shape, generator=gen, dtype=torch.float32)
+        x = torch.randn(shape, generator=gen, dtype=torch.float32)
         if spec.init == "ones":
             out[name] = norm_center + x * norm_std
         elif std_by_fan_in and spec.fan_in > 0:
