@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
                     [--shape 135m|360m|1.7b] [--batch B] [--context C] [--layers L] [--skip-points]
-                    [--skip-e2e] [--designs s,m [--only-design llama,nafezen,tazadra,sedopel,selovik]]
+                    [--skip-e2e] [--designs s,m [--only-design llama,nafezen,tazadra,sedopel,selovik,setenex]]
 
 A step is one decode step of a batch of 8 sequences whose context ends at 4,096
 tokens (prompt 2,048 + 2,048 decoded); ``value`` is decoded tokens per second,
@@ -236,10 +236,10 @@ def timeline(engine, batch, path, rng, vocab):
 
 
 # ---------------------------------------------------------------------------
-# --designs: the Nafezen, Tazadra, Sedopel and Selovik designs beside the Llama decoder at equal width and depth
+# --designs: the Nafezen, Tazadra, Sedopel, Selovik and Setenex designs beside the Llama decoder at equal width and depth
 # ---------------------------------------------------------------------------
 def design_configs(size: str):
-    """(Llama, Nafezen, Tazadra, Sedopel, Selovik) configurations of one width, depth, vocabulary and dense
+    """(Llama, Nafezen, Tazadra, Sedopel, Selovik, Setenex) configurations of one width, depth, vocabulary and dense
     feed-forward size; the Nafezen layers alternate latent attention with dense and expert
     feed-forwards and hold one retention layer in four; the Tazadra layers are attention with a
     sink + dense, WKV + experts, selective scan + experts, and attention that reads the first
@@ -247,7 +247,10 @@ def design_configs(size: str):
     attention beside lightning attention) + dense with the gated delta rule, which has a dense
     feed-forward every other time; the Selovik layers are differential attention (two maps of half a
     head's size over values of a head's size, a window of 1,024) with dense and expert feed-forwards
-    in turn, six layers of which the second and third run twice (eight layer runs)."""
+    in turn, six layers of which the second and third run twice (eight layer runs); the Setenex layers
+    alternate attention with a bias per distance (a window of 1,024 that keeps 64 first tokens) and latent
+    attention with queries straight from the input and a window of 1,024, all with experts, six layers
+    of which the second and third run twice."""
     width, heads, ff, layers, q_rank, kv_rank, experts, top = {
         "s": (1024, 16, 2816, 8, 384, 256, 16, 2),
         "m": (2048, 16, 5632, 8, 768, 512, 32, 4),
@@ -308,10 +311,20 @@ def design_configs(size: str):
     selovik = {"architecture": "Selovik", "vocab": 32768, "width": width, "norm": {"eps": 1e-5},
                "embedding": {"scale": 1.0, "bigram": {"buckets": 8191, "mul_prev": 31, "mul_cur": 17}},
                "logit_scale": 1.0, "loop": {"start": 1, "stop": 3, "times": 2}, "layers": v_layers}
-    return llama, nafezen, tazadra, sedopel, selovik
+    biased = {"heads": heads, "kv_heads": heads // 4, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "bias_max": 1024,
+              "mask": {"size": 1024, "keep_first": 64}}
+    direct = {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "kv_rank": kv_rank,
+              "rot": {"base": 10000.0, "dims": dim // 2}, "scale": (dim + dim // 2) ** -0.5, "mask": {"size": 1024}}
+    x_moe = {"kind": "moe", "expert": {"ff": ff // (2 * top)},
+             "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}}
+    x_layers = [{"type": "attention" if i % 2 == 0 else "latent_attention", "mixer": biased if i % 2 == 0 else direct,
+                 "mlp": x_moe} for i in range(layers - 2)]
+    setenex = {"architecture": "Setenex", "vocab": 32768, "width": width, "norm": {"eps": 1e-5},
+               "embedding": {"scale": 1.0}, "loop": {"start": 1, "stop": 3, "times": 2}, "layers": x_layers}
+    return llama, nafezen, tazadra, sedopel, selovik, setenex
 
 
-DESIGN_NAMES = ("llama", "nafezen", "tazadra", "sedopel", "selovik")
+DESIGN_NAMES = ("llama", "nafezen", "tazadra", "sedopel", "selovik", "setenex")
 
 
 def profile_steps(args) -> int:
@@ -456,7 +469,7 @@ def compare_designs(args) -> int:
                 for part in engine.model.blocks[entry.layer].parts():
                     if hasattr(part, "step_bytes"):
                         weight_bytes += part.step_bytes(batch) - part.parameter_bytes()
-            step_bytes = weight_bytes + batch * (context - steps / 2) * engine.cache.kv_bytes_per_token()
+            step_bytes = weight_bytes + batch * engine.cache.kv_bytes_read(context - steps // 2)
             for s in slots:
                 engine.release_slot(s)
             print(json.dumps({
@@ -498,10 +511,10 @@ def main() -> int:
     ap.add_argument("--shape", default="135m", choices=sorted(SHAPES),
                     help="layer sizes: the SmolLM2-135M shape (the benchmark) or a larger one of the family")
     ap.add_argument("--designs", metavar="SIZES", default=None,
-                    help="instead of the benchmark: the Nafezen, Tazadra, Sedopel and Selovik designs beside the Llama decoder at "
+                    help="instead of the benchmark: the Nafezen, Tazadra, Sedopel, Selovik and Setenex designs beside the Llama decoder at "
                          "equal width and depth, sizes 's' and/or 'm' with commas: prefill, its parts, decoding")
     ap.add_argument("--only-design", metavar="NAMES", default=None,
-                    help="with --designs: only these of llama, nafezen, tazadra, sedopel, selovik (commas between them)")
+                    help="with --designs: only these of llama, nafezen, tazadra, sedopel, selovik, setenex (commas between them)")
     ap.add_argument("--profile-steps", type=int, default=0,
                     help="with --designs: run this many eager prompt and decode steps of one design's first "
                          "four layers for a profiler instead of the timed comparison")

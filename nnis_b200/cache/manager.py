@@ -320,6 +320,12 @@ class CacheManager:
         return sum(len(g.entries) * g.kv_heads * (g.head_dim + g.value_dim) * g.k.element_size()
                    for g in self.groups)
 
+    def kv_bytes_read(self, length: int) -> int:
+        """Bytes of keys and values that one more token of a sequence of ``length`` positions reads over all
+        layers: a windowed group's window and kept first positions, the whole of another's."""
+        return sum(len(g.entries) * g.kv_heads * (g.head_dim + g.value_dim) * g.k.element_size()
+                   * (min(length, g.window + g.keep_first) if g.window > 0 else length) for g in self.groups)
+
     # -- telemetry (crates/nnis-rt/src/kv_telemetry.rs:42-80) ----------------
     def usage(self) -> Dict[str, object]:
         return {

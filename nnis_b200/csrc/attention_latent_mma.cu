@@ -174,8 +174,9 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
             for (int j = 0; j < KB; ++j)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    int key = tk + j * 8 + c_lo + (e & 1);
-                    float v = key <= pos_r[e >> 1] && key > pos_r[e >> 1] - reach ? s[j][e] * sc : -INFINITY;
+                    // (one comparison for both ends: a key ahead of the row wraps to a large number)
+                    const unsigned back = (unsigned)(pos_r[e >> 1] - (tk + j * 8 + c_lo + (e & 1)));
+                    float v = back < (unsigned)reach ? s[j][e] * sc : -INFINITY;
                     s[j][e] = v;
                     mx[e >> 1] = fmaxf(mx[e >> 1], v);
                 }

@@ -337,6 +337,9 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
     const int h0 = hk * G;  // the group's first query head
     const int pos = token_pos[n];
     float* qs = q_smem + (size_t)warp * G * dk;
+    // which of the head's values a lane holds: neighbours where its share is whole (one load a row), else every 32nd
+    const bool vec = R == 4 && dv == 128;
+    auto place = [&](int r) { return vec ? lane * R + r : lane + 32 * r; };
 
     float m[G], l[G], acc[G][R];
 #pragma unroll
@@ -420,17 +423,25 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
             // the value rows of several keys are asked for together (beyond the last key: the last row
             // again, with a weight of zero)
             const int count = min(32, end - c);
-            constexpr int TOGETHER = R >= 4 ? 4 : 8;
+            constexpr int TOGETHER = 8;
             for (int j0 = 0; j0 < count; j0 += TOGETHER) {
                 float vr[TOGETHER][R];
 #pragma unroll
                 for (int u = 0; u < TOGETHER; ++u) {
                     const int rj = __shfl_sync(0xffffffffu, row_index, min(j0 + u, count - 1));
                     const T* vrow = v_cache + (size_t)rj * dv;
+                    if (R == 4 && vec) {
+                        const float4 v4 = load4(vrow + lane * 4);
+                        vr[u][0] = v4.x;
+                        vr[u][1 % R] = v4.y;
+                        vr[u][2 % R] = v4.z;
+                        vr[u][3 % R] = v4.w;
+                    } else {
 #pragma unroll
-                    for (int r = 0; r < R; ++r) {
-                        int i = lane + 32 * r;
-                        vr[u][r] = i < dv ? to_float(vrow[i]) : 0.f;
+                        for (int r = 0; r < R; ++r) {
+                            int i = lane + 32 * r;
+                            vr[u][r] = i < dv ? to_float(vrow[i]) : 0.f;
+                        }
                     }
                 }
 #pragma unroll
@@ -455,7 +466,7 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
             T* o = out + ((size_t)n * nq + hq) * dv;
 #pragma unroll
             for (int r = 0; r < R; ++r) {
-                int i = lane + 32 * r;
+                const int i = place(r);
                 if (i < dv) o[i] = from_float<T>(acc[g][r] * inv * (ge ? ge[i] : 1.0f));
             }
         } else {
@@ -466,7 +477,7 @@ attn_sink_group_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, c
             }
 #pragma unroll
             for (int r = 0; r < R; ++r) {
-                int i = lane + 32 * r;
+                const int i = place(r);
                 if (i < dv) rec[2 + i] = acc[g][r];
             }
         }

@@ -25,7 +25,7 @@ constexpr int kSinkStages = 3;
 
 // DK, DV: sizes in shared memory; PAD: the heads hold fewer values (dk, dv); BIAS: a bias per distance
 template <int DK, int DV, bool PAD, bool BIAS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, (DK <= 64 && DV <= 64) ? 3 : 1)
 attn_sink_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache,
                      const bf16* __restrict__ v_cache, const int* __restrict__ tiles,
                      const int* __restrict__ seq_first_row, const int* __restrict__ seq_start,
@@ -122,6 +122,9 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cach
         lo_r[h] = window > 0 ? pos_r[h] - window + 1 : 0;
         if (chunk > 0) lo_r[h] = max(lo_r[h], (pos_r[h] / chunk) * chunk);
     }
+    // the first key of the warp's last row, the largest of its rows'
+    int warp_hi_lo = window > 0 ? pos0 + warp * 16 + 15 - window + 1 : 0;
+    if (chunk > 0) warp_hi_lo = max(warp_hi_lo, ((pos0 + warp * 16 + 15) / chunk) * chunk);
     float o[NT][4];
 #pragma unroll
     for (int j = 0; j < NT; ++j)
@@ -148,6 +151,8 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cach
             if (chunk > 0 && t0 + kSinkPage <= ((pos0 + warp * 16) / chunk) * chunk) continue;
             if (window > 0 && t0 + kSinkPage <= pos0 + warp * 16 - window + 1) continue;
         }
+        // every row of the warp sees every key of the page (most pages of a long walk): no mask
+        const bool full = t0 + kSinkPage - 1 <= pos0 + warp * 16 && (t0 >= warp_hi_lo || t0 + kSinkPage <= keep);
         // the biases, times log2(e), of the distances that this thread's scores of the page lie on:
         // row r_lo + 8 h against key 8 j + c_lo + e is the distance (of the warp's first row) + r_lo -
         // c_lo + 8 (h - j) - e, so h - j = -7 .. 1 and e = 0, 1
@@ -183,8 +188,6 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cach
         for (int j = 0; j < 8; ++j)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                int key = t0 + j * 8 + c_lo + (e & 1);
-                bool ok = key <= pos_r[e >> 1] && (key >= lo_r[e >> 1] || key < keep);
                 float v;
                 if (cap > 0.f) {  // cap * tanh(x / cap) = cap * (1 - 2 / (exp(2 x / cap) + 1))
                     float e2 = exp2f(s[j][e] * scale * cap_in);
@@ -193,10 +196,22 @@ attn_sink_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cach
                     v = s[j][e] * sc;
                 }
                 if (BIAS) v += near[(e >> 1) - j + 7][e & 1];
-                v = ok ? v : -INFINITY;
                 s[j][e] = v;
-                mx[e >> 1] = fmaxf(mx[e >> 1], v);
             }
+        if (!full) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int key = t0 + j * 8 + c_lo + (e & 1);
+                    const bool ok = key <= pos_r[e >> 1] && (key >= lo_r[e >> 1] || key < keep);
+                    s[j][e] = ok ? s[j][e] : -INFINITY;
+                }
+        }
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) mx[e >> 1] = fmaxf(mx[e >> 1], s[j][e]);
         float alpha[2], base[2];
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
