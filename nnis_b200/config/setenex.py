@@ -190,7 +190,7 @@ class SetenexConfig:
                 "vdim": m["vdim"], "scale": m["scale"], "window": window,
                 "keep_first": min(m["mask"]["keep_first"], MAX_POSITIONS),
                 "distance_bias": {"far": m["bias_max"], "rows": RANDOM_TABLE_ROWS}, "qk_norm": "head_weight",
-                "eps": self.norm_eps,
+                "eps": self.norm_eps, "pad_heads": True,
                 # no rotation: a position shows in the distance bias alone
                 "position": PartSpec("rope_frequencies", {"dims": 0, "base": 1.0, "pairing": "half"}), "leaf": "",
                 "names": {"q": "mix.q", "k": "mix.k", "v": "mix.v", "o": "mix.o", "q_norm": "mix.q.norm",

@@ -36,12 +36,12 @@ part has no k/v projection, norm or cache of its own and reads another schedule 
 One projection makes q, k, v and the gate's logits in float32 (their matrices are
 stacked at load); ``qkv_prep`` norms, rotates, stores and takes the sigmoid; the attention
 kernel serves prompts, later portions and single tokens alike; prompt steps in bfloat16 with
-key and value heads of up to 128 values (multiples of eight) run a tensor-core form of it
-(``attention_sink_mma``).
+key and value heads of 64 or of 128 run a tensor-core form of it (``attention_sink_mma``); with
+``pad_heads`` so do other sizes up to 128 in multiples of eight, padded with zeros in shared memory.
 
 params: hidden_size, heads, kv_heads, dim, vdim, scale, softcap, chunk, window, keep_first,
 distance_bias, sink, gate, qk_norm, head_scale, eps, position (a ``rope_frequencies`` PartSpec),
-kv ("own" | "shared"), names {q, k, v, o, q_norm, k_norm, sink, gate, head_scale, distance_bias}.
+pad_heads, kv ("own" | "shared"), names {q, k, v, o, q_norm, k_norm, sink, gate, head_scale, distance_bias}.
 """
 from __future__ import annotations
 
@@ -116,6 +116,7 @@ class SinkAttention(Part):
         self.qk_norm = bool(norm) and not self.head_norm and not self.head_weight_norm
         self.has_head_scale = bool(params.get("head_scale", False))
         self.eps = float(params.get("eps", 1e-6))
+        self.pad_heads = bool(params.get("pad_heads", False))
         self.own_kv = params.get("kv", "own") == "own"
         self.names = params["names"]
         if self.heads % self.kv_heads:
@@ -218,7 +219,9 @@ class SinkAttention(Part):
     TILES_64 = "prefill_mma/tiles64"  # (sequence, first query) per 64 queries of the step
 
     def _mma_prompt(self) -> bool:
-        return self.dtype == torch.bfloat16 and ops.attention_sink_mma_takes(self.dim, self.vdim, PAGE_SIZE)
+        whole = self.dim == self.vdim and self.dim in (64, 128)
+        return self.dtype == torch.bfloat16 and (whole or self.pad_heads) \
+            and ops.attention_sink_mma_takes(self.dim, self.vdim, PAGE_SIZE)
 
     def step_tables(self, counts, starts, have=()):
         """The 64-query tiles of the tensor-core prompt kernel (the same list for every layer)."""
