@@ -20,6 +20,7 @@ from .sedopel import SedopelConfig
 from .selovik import SelovikConfig
 from .setenex import SetenexConfig
 from .tazadra import TazadraConfig
+from .zadurax import ZaduraxConfig
 from .spec import ModelSpec
 
 _ARCHITECTURES: Dict[str, Type] = {}
@@ -89,3 +90,4 @@ register_architecture(TazadraConfig.architecture, TazadraConfig)
 register_architecture(SedopelConfig.architecture, SedopelConfig)
 register_architecture(SelovikConfig.architecture, SelovikConfig)
 register_architecture(SetenexConfig.architecture, SetenexConfig)
+register_architecture(ZaduraxConfig.architecture, ZaduraxConfig)

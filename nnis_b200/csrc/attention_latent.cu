@@ -12,14 +12,16 @@
 //                    the float32 row [q (H x (plain | rotated)) | c raw | kr raw | gate (H)] ->
 //                    q's plain parts packed (operand dtype), its rotated parts turned and put
 //                    behind the latent's place in the packed query rows, normed c and turned kr
-//                    into the cache row, the sigmoid of the gate's logits
+//                    into the cache row, the sigmoid of the gate's logits; `magnitude` multiplies every
+//                    cosine and sine
 //                    (both: pairs (i, i + dims / 2), or with `neighbours` (2i, 2i + 1))
 //   attention_latent one warp per (query token, head) walks the visible rows 32 at a
 //                    time with an online softmax in float32; prompts and single
 //                    tokens, float32 and bfloat16 storage, any sizes; the key range
 //                    may be split over several warps (records merged in order); with
 //                    `window` a query at position p sees keys above p - window only; the
-//                    output may be multiplied by a gate per (token, head)
+//                    output may be multiplied by a gate per (token, head); with `sink` the softmax's
+//                    denominator also holds exp(sink[head]) (counted in the first slice)
 #include <float.h>
 
 #include "attention_merge.cuh"
@@ -90,7 +92,7 @@ latent_prep_direct_kernel(const float* __restrict__ a, const float* __restrict__
                           const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                           const int* __restrict__ page_table, int table_cols, T* __restrict__ q_plain,
                           T* __restrict__ q_rows, T* __restrict__ cache, float* __restrict__ gate, int heads, int dim,
-                          int kv_rank, int rot, int rot_dims, int page_size, float eps, int neighbours, int a_cols) {
+                          int kv_rank, int rot, int rot_dims, int page_size, float eps, int neighbours, int a_cols, float magnitude) {
     extern __shared__ float turn[];
     __shared__ float sums[8];
     pdl_wait();
@@ -103,7 +105,12 @@ latent_prep_direct_kernel(const float* __restrict__ a, const float* __restrict__
     const float* c = row + nq;
     float* cs = turn;
     float* sn = turn + max(half, 1);
-    for (int j = tid; j < half; j += 256) sincosf((float)pos * freq[j], sn + j, cs + j);
+    for (int j = tid; j < half; j += 256) {
+        float s, co;
+        sincosf((float)pos * freq[j], &s, &co);
+        sn[j] = s * magnitude;
+        cs[j] = co * magnitude;
+    }
     float ss = 0.f;
     for (int i = tid; i < kv_rank; i += 256) ss = fmaf(c[i], c[i], ss);
     ss = warp_sum(ss);
@@ -150,7 +157,7 @@ latent_warp_kernel(const T* __restrict__ q, const T* __restrict__ cache,
                    const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                    const int* __restrict__ page_table, int table_cols, T* __restrict__ out,
                    float* __restrict__ partial, int n_tokens, int heads, int dk, int dv,
-                   int page_size, float scale, int n_splits, int window, const float* __restrict__ gate) {
+                   int page_size, float scale, int n_splits, int window, const float* __restrict__ gate, const float* __restrict__ sink) {
     extern __shared__ float q_smem[];
     int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     int n = blockIdx.x * 4 + warp;
@@ -172,6 +179,10 @@ latent_warp_kernel(const T* __restrict__ q, const T* __restrict__ cache,
         per = (per + 31) & ~31;
         int start = lo + split * per;
         int end = min(hi, start + per);
+        if (sink && split == 0) {  // a score without a key and without a value
+            m = sink[h];
+            l = 1.f;
+        }
         const int* table = page_table + (size_t)token_seq[n] * table_cols;
         for (int c0 = start; c0 < end; c0 += 32) {
             int t = c0 + lane;
@@ -232,13 +243,13 @@ template <typename T>
 static int launch_latent(const void* q, const void* cache, const int* token_pos, const int* token_seq,
                          const int* page_table, int table_cols, void* out, float* partial,
                          int n_tokens, int heads, int dk, int dv, int page_size, float scale,
-                         int n_splits, int window, const float* gate, cudaStream_t stream) {
+                         int n_splits, int window, const float* gate, const float* sink, cudaStream_t stream) {
     dim3 grid((n_tokens + 3) / 4, heads, n_splits);
     size_t smem = 4 * (size_t)dk * sizeof(float);
 #define NNIS_LATENT_CASE(R) \
     latent_warp_kernel<T, R><<<grid, 128, smem, stream>>>( \
         (const T*)q, (const T*)cache, token_pos, token_seq, page_table, table_cols, (T*)out, partial, \
-        n_tokens, heads, dk, dv, page_size, scale, n_splits, window, gate)
+        n_tokens, heads, dk, dv, page_size, scale, n_splits, window, gate, sink)
     if (dv <= 32) NNIS_LATENT_CASE(1);
     else if (dv <= 64) NNIS_LATENT_CASE(2);
     else if (dv <= 128) NNIS_LATENT_CASE(4);
@@ -289,7 +300,7 @@ NNIS_API int nnis_latent_prep_direct(const float* a, const float* wkv, const flo
                                      const int* token_seq, const int* page_table, int table_cols, void* q_plain,
                                      void* q_rows, void* cache, float* gate, int n_tokens, int heads, int dim,
                                      int kv_rank, int rot, int rot_dims, int page_size, float eps, int neighbours,
-                                     int a_cols, int dtype, cudaStream_t stream) {
+                                     int a_cols, float magnitude, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || heads <= 0 || dim <= 0 || kv_rank <= 0 || rot < 0 || rot_dims < 0 || (rot_dims & 1) ||
         rot_dims > rot || page_size <= 0 || table_cols <= 0 || !(eps > 0.f) || !a || !wkv || !freq || !q_plain ||
         !q_rows || !cache || !token_pos || !token_seq || !page_table)
@@ -301,11 +312,11 @@ NNIS_API int nnis_latent_prep_direct(const float* a, const float* wkv, const flo
     if (dtype == NNIS_DTYPE_F32)
         e = launch_dependent(latent_prep_direct_kernel<float>, n_tokens, 256, smem, stream, a, wkv, freq, token_pos,
                              token_seq, page_table, table_cols, (float*)q_plain, (float*)q_rows, (float*)cache, gate,
-                             heads, dim, kv_rank, rot, rot_dims, page_size, eps, neighbours, a_cols);
+                             heads, dim, kv_rank, rot, rot_dims, page_size, eps, neighbours, a_cols, magnitude);
     else if (dtype == NNIS_DTYPE_BF16)
         e = launch_dependent(latent_prep_direct_kernel<bf16>, n_tokens, 256, smem, stream, a, wkv, freq, token_pos,
                              token_seq, page_table, table_cols, (bf16*)q_plain, (bf16*)q_rows, (bf16*)cache, gate,
-                             heads, dim, kv_rank, rot, rot_dims, page_size, eps, neighbours, a_cols);
+                             heads, dim, kv_rank, rot, rot_dims, page_size, eps, neighbours, a_cols, magnitude);
     else
         return NNIS_ERR_UNSUPPORTED;
     return e == cudaSuccess ? NNIS_OK : (int)e;
@@ -313,12 +324,12 @@ NNIS_API int nnis_latent_prep_direct(const float* a, const float* wkv, const flo
 
 // Scratch: `partial` needs n_tokens * heads * n_splits * (dv + 2) floats when
 // n_splits > 1 and may be null otherwise.  `window` 0: every key up to the query's; `gate`:
-// float32 [n_tokens, heads] or null.
+// float32 [n_tokens, heads] or null; `sink`: float32 [heads] or null.
 NNIS_API int nnis_attention_latent(const void* q, const void* cache, const int* token_pos,
                                    const int* token_seq, const int* page_table, int table_cols,
                                    void* out, float* partial, int n_tokens, int heads, int dk, int dv,
                                    int page_size, float scale, int n_splits, int window, const float* gate,
-                                   int dtype, cudaStream_t stream) {
+                                   const float* sink, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || heads <= 0 || dk <= 0 || dv <= 0 || dv > dk || page_size <= 0 ||
         table_cols <= 0 || n_splits <= 0 || window < 0)
         return NNIS_ERR_ARGUMENT;
@@ -326,9 +337,9 @@ NNIS_API int nnis_attention_latent(const void* q, const void* cache, const int* 
     if (n_splits > 1 && !partial) return NNIS_ERR_ARGUMENT;
     if (dtype == NNIS_DTYPE_F32)
         return launch_latent<float>(q, cache, token_pos, token_seq, page_table, table_cols, out, partial,
-                                    n_tokens, heads, dk, dv, page_size, scale, n_splits, window, gate, stream);
+                                    n_tokens, heads, dk, dv, page_size, scale, n_splits, window, gate, sink, stream);
     if (dtype == NNIS_DTYPE_BF16)
         return launch_latent<bf16>(q, cache, token_pos, token_seq, page_table, table_cols, out, partial,
-                                   n_tokens, heads, dk, dv, page_size, scale, n_splits, window, gate, stream);
+                                   n_tokens, heads, dk, dv, page_size, scale, n_splits, window, gate, sink, stream);
     return NNIS_ERR_UNSUPPORTED;
 }

@@ -15,7 +15,8 @@
 //
 // With `window` a query at position p sees keys above p - window only, and the walk begins at
 // the page of the first key that the tile's first row sees.  `gate` (float32, one per stacked
-// row) multiplies the row's output.
+// row) multiplies the row's output.  With `sink` (float32 [heads]) the softmax's denominator also holds
+// exp(sink[head]), counted in the first slice.
 //
 // The key range may be cut into slices (blockIdx.z), for steps with few rows and long
 // contexts: a slice leaves [max, sum, unnormalised output] per row and the merge kernel
@@ -44,7 +45,8 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
                   const int* __restrict__ token_pos, const int* __restrict__ token_seq,
                   const int* __restrict__ page_table, int table_cols, bf16* __restrict__ out,
                   float* __restrict__ partial, int heads, int dk, int dv, int dkp, int tiles_per_token,
-                  float scale, int n_splits, int window, const float* __restrict__ gate) {
+                  float scale, int n_splits, int window, const float* __restrict__ gate,
+                  const float* __restrict__ sink) {
     constexpr int KH = NT == 16 ? 64 : 32, KB = KH / 8, RUN = NT * 8;
     constexpr int TILE = SPLIT_ROWS ? 2 * kLatRows : kLatRows;  // rows of the CTA
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -134,6 +136,13 @@ latent_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache,
 #pragma unroll
         for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+    if (sink && split == 0) {  // a score without a key and without a value (its sum counted in one lane of four)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            m_run[h] = sink[(r0 + g_row + warp * 16 + r_lo + h * 8) % heads] * kLog2e;
+            l_run[h] = (lane & 3) == 0 ? 1.f : 0.f;
+        }
+    }
     const float sc = scale * kLog2e;
     const int KS = dkp >> 4;
 
@@ -302,13 +311,13 @@ NNIS_API int nnis_attention_latent_mma_tile_rows(int dv) { return latent_tile_ro
 // null, and then every row of the step is one token of a sequence of its own (n_tokens
 // rows, ceil(heads / tile rows) tiles each).
 // `partial`: float32 [n_tokens * heads * n_splits * (dv + 2)] when n_splits > 1.  `gate`: float32
-// [n_tokens, heads] or null.
+// [n_tokens, heads] or null; `sink`: float32 [heads] or null.
 NNIS_API int nnis_attention_latent_mma(const void* q, const void* cache, const int* tiles, int n_tiles,
                                        const int* seq_first_row, const int* seq_start,
                                        const int* seq_count, const int* token_pos, const int* token_seq,
                                        const int* page_table, int table_cols, void* out, float* partial,
                                        int n_tokens, int heads, int dk, int dv, int page_size,
-                                       float scale, int n_splits, int window, const float* gate,
+                                       float scale, int n_splits, int window, const float* gate, const float* sink,
                                        cudaStream_t stream) {
     if (n_tokens <= 0 || heads <= 0 || table_cols <= 0 || n_splits <= 0 || window < 0 || !q || !cache || !out ||
         !page_table)
@@ -329,7 +338,7 @@ NNIS_API int nnis_attention_latent_mma(const void* q, const void* cache, const i
     const size_t smem = latent_mma_smem(dk, dv, stages);
     using Kernel = void (*)(const bf16*, const bf16*, const int*, const int*, const int*, const int*, const int*,
                             const int*, const int*, int, bf16*, float*, int, int, int, int, int, float, int, int,
-                            const float*);
+                            const float*, const float*);
     Kernel kernel;
     if (run == 128) kernel = stages == 3 ? latent_mma_kernel<3, 16, true> : latent_mma_kernel<2, 16, true>;
     else if (split_rows) kernel = stages == 3 ? latent_mma_kernel<3, 32, true> : latent_mma_kernel<2, 32, true>;
@@ -341,7 +350,7 @@ NNIS_API int nnis_attention_latent_mma(const void* q, const void* cache, const i
     cudaError_t e = launch_dependent(kernel, grid, 256, smem, stream, (const bf16*)q, (const bf16*)cache, tiles,
                                      seq_first_row, seq_start, seq_count, token_pos, token_seq, page_table,
                                      table_cols, (bf16*)out, partial, heads, dk, dv, dkp, tiles_per_token, scale,
-                                     n_splits, window, gate);
+                                     n_splits, window, gate, sink);
     if (e != cudaSuccess) return (int)e;
     if (n_splits > 1) {
         size_t rows = (size_t)n_tokens * heads;

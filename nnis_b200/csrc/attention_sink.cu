@@ -17,7 +17,8 @@
 //                   (one per head, or one per output value).  A head may hold `maps` vectors of equal
 //                   size side by side (the queries and keys of several attention maps over one set of
 //                   values); each is turned by itself over its own first `rot` values.  `magnitude`
-//                   multiplies every cosine and sine (1: a pure rotation).
+//                   multiplies every cosine and sine (1: a pure rotation).  With `v_is_k` the rows have no v
+//                   columns: the values are the keys as projected, before norm and rotation.
 //   attn_sink       one warp per (query token, query head) walks the visible keys 32 at a time with
 //                   an online softmax in float32: score = cap * tanh(scale * q.k / cap) (cap 0: none);
 //                   a query at position p sees keys j <= p with j >= p - window + 1 (window > 0) and
@@ -126,7 +127,7 @@ qkv_prep_heads_kernel(const float* __restrict__ a, const float* __restrict__ wq,
                       const int* __restrict__ token_seq, const int* __restrict__ page_table, int table_cols,
                       T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
                       float* __restrict__ gate_out, int H, int G, int dk, int dv, int rot, int pairing,
-                      int norm_heads, int gate_cols, int page_size, float eps, int maps, float magnitude) {
+                      int norm_heads, int gate_cols, int page_size, float eps, int maps, float magnitude, int v_is_k) {
     extern __shared__ float turned[];  // [8 warps][dk]
     pdl_wait();
     pdl_launch_dependents();
@@ -135,7 +136,9 @@ qkv_prep_heads_kernel(const float* __restrict__ a, const float* __restrict__ wq,
     if (pos < 0) return;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int nq = H * dk, nk = G * dk, nv = G * dv;
-    const float* row = a + (size_t)n * (nq + nk + nv + gate_cols);
+    const int v_off = v_is_k ? nq : nq + nk;  // (values that are the keys as projected: no columns of their own)
+    const int gate_off = v_off + nv;
+    const float* row = a + (size_t)n * (gate_off + gate_cols);
     const float p = (float)pos;
     const int half = rot >> 1;
     const int sub = dk / maps;  // the size of one map's vector
@@ -197,10 +200,10 @@ qkv_prep_heads_kernel(const float* __restrict__ a, const float* __restrict__ wq,
     }
     for (int i = threadIdx.x; i < nv; i += 256) {
         const int head = i / dv, within = i - head * dv;
-        v_cache[(cache_row + (size_t)head * page_size) * dv + within] = from_float<T>(row[nq + nk + i]);
+        v_cache[(cache_row + (size_t)head * page_size) * dv + within] = from_float<T>(row[v_off + i]);
     }
     for (int i = threadIdx.x; i < gate_cols; i += 256)
-        gate_out[(size_t)n * gate_cols + i] = 1.0f / (1.0f + expf(-row[nq + nk + nv + i]));
+        gate_out[(size_t)n * gate_cols + i] = 1.0f / (1.0f + expf(-row[gate_off + i]));
 }
 
 // partial record per (token, head, slice): [0] running max, [1] running sum, [2 .. 2 + dv) output
@@ -627,11 +630,11 @@ NNIS_API int nnis_qkv_prep_heads(const float* a, const float* wq, const float* w
                                  const float* freq, const int* token_pos, const int* token_seq, const int* page_table, int table_cols, void* q_out,
                                  void* k_cache, void* v_cache, float* gate_out, int n_tokens, int H, int G, int dk,
                                  int dv, int rot, int pairing, int norm_heads, int gate_cols, int page_size,
-                                 float eps, int maps, float magnitude, int dtype, cudaStream_t stream) {
+                                 float eps, int maps, float magnitude, int v_is_k, int dtype, cudaStream_t stream) {
     if (n_tokens <= 0 || H <= 0 || G < 0 || dk <= 0 || dv <= 0 || rot < 0 || gate_cols < 0 || !a || !q_out ||
         !token_pos)
         return NNIS_ERR_ARGUMENT;
-    if (maps <= 0 || dk % maps) return NNIS_ERR_ARGUMENT;
+    if (maps <= 0 || dk % maps || (v_is_k && dk != dv)) return NNIS_ERR_ARGUMENT;
     if ((rot & 1) || rot > dk / maps || dk > 1024 || ((dk / maps) & 1 && maps > 1 && !pairing))
         return NNIS_ERR_UNSUPPORTED;
     if (rot > 0 && !freq) return NNIS_ERR_ARGUMENT;
@@ -643,12 +646,12 @@ NNIS_API int nnis_qkv_prep_heads(const float* a, const float* wq, const float* w
         e = launch_dependent(qkv_prep_heads_kernel<float>, (unsigned)n_tokens, 256, smem, stream, a, wq, wk, q_scale,
                              freq, token_pos, token_seq, page_table, table_cols, (float*)q_out, (float*)k_cache,
                              (float*)v_cache, gate_out, H, G, dk, dv, rot, pairing, norm_heads, gate_cols, page_size,
-                             eps, maps, magnitude);
+                             eps, maps, magnitude, v_is_k);
     else if (dtype == NNIS_DTYPE_BF16)
         e = launch_dependent(qkv_prep_heads_kernel<bf16>, (unsigned)n_tokens, 256, smem, stream, a, wq, wk, q_scale,
                              freq, token_pos, token_seq, page_table, table_cols, (bf16*)q_out, (bf16*)k_cache,
                              (bf16*)v_cache, gate_out, H, G, dk, dv, rot, pairing, norm_heads, gate_cols, page_size,
-                             eps, maps, magnitude);
+                             eps, maps, magnitude, v_is_k);
     else
         return NNIS_ERR_UNSUPPORTED;
     return e == cudaSuccess ? NNIS_OK : (int)e;

@@ -4,6 +4,8 @@
 // consecutive [N, K] matrices.  Latent attention uses it twice: to carry the
 // queries into the latent space (W = the keys' up-projection, transposed per head at
 // load) and to carry the attention's latent output to the heads' values.
+// With `gate` (float32 logits, row stride gate_ld, column b * N + n for output n of head b) a sum is
+// multiplied by the sigmoid of its logit before it is rounded.
 // Operands float32 or bfloat16, float32 accumulation with fmaf on the CUDA cores
 // (the float32 path, and the bfloat16 path of shapes the tensor-core kernel refuses).
 #include "async_copy.cuh"
@@ -11,11 +13,15 @@
 
 namespace nnis {
 
+__device__ __forceinline__ float gated(float v, const float* gate, long long gate_ld, int m, int col) {
+    return gate ? v * (1.0f / (1.0f + expf(-gate[(size_t)m * gate_ld + col]))) : v;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 batched_linear_kernel(const T* __restrict__ A, long long lda, long long a_bs,
                       const T* __restrict__ W, T* __restrict__ C, long long ldc, long long c_bs,
-                      int M, int N, int K) {
+                      int M, int N, int K, const float* __restrict__ gate, long long gate_ld) {
     constexpr int BM = 64, BN = 64, BK = 16, PAD = 4;
     __shared__ __align__(16) float As[BK][BM + PAD];
     __shared__ __align__(16) float Ws[BK][BN + PAD];
@@ -54,7 +60,7 @@ batched_linear_kernel(const T* __restrict__ A, long long lda, long long a_bs,
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             int n = n0 + tx * 4 + j;
-            if (n < N) C[(size_t)m * ldc + n] = from_float<T>(acc[i][j]);
+            if (n < N) C[(size_t)m * ldc + n] = from_float<T>(gated(acc[i][j], gate, gate_ld, m, b * N + n));
         }
     }
 }
@@ -64,7 +70,8 @@ batched_linear_kernel(const T* __restrict__ A, long long lda, long long a_bs,
 template <typename T>
 __global__ void __launch_bounds__(256)
 batched_rows_kernel(const T* __restrict__ A, long long lda, long long a_bs, const T* __restrict__ W,
-                    T* __restrict__ C, long long ldc, long long c_bs, int M, int N, int K) {
+                    T* __restrict__ C, long long ldc, long long c_bs, int M, int N, int K,
+                    const float* __restrict__ gate, long long gate_ld) {
     pdl_wait();
     pdl_launch_dependents();
     int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -103,24 +110,25 @@ batched_rows_kernel(const T* __restrict__ A, long long lda, long long a_bs, cons
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
         float v = warp_sum(acc[i]);
-        if (lane == 0 && m0 + i < M) C[(size_t)(m0 + i) * ldc + (size_t)b * c_bs + n] = from_float<T>(v);
+        if (lane == 0 && m0 + i < M)
+            C[(size_t)(m0 + i) * ldc + (size_t)b * c_bs + n] = from_float<T>(gated(v, gate, gate_ld, m0 + i, b * N + n));
     }
 }
 
 template <typename T>
 static int launch_batched(const void* A, long long lda, long long a_bs, const void* W, void* C,
-                          long long ldc, long long c_bs, int batch, int M, int N, int K,
-                          cudaStream_t stream) {
+                          long long ldc, long long c_bs, int batch, int M, int N, int K, const float* gate,
+                          long long gate_ld, cudaStream_t stream) {
     if (M <= 16) {
         dim3 grid((N + 7) / 8, (M + 7) / 8, batch);
         cudaError_t e = launch_dependent(batched_rows_kernel<T>, grid, 256, 0, stream, (const T*)A, lda, a_bs,
-                                         (const T*)W, (T*)C, ldc, c_bs, M, N, K);
+                                         (const T*)W, (T*)C, ldc, c_bs, M, N, K, gate, gate_ld);
         return e == cudaSuccess ? NNIS_OK : (int)e;
     } else {
         dim3 grid((N + 63) / 64, (M + 63) / 64, batch);
         if (grid.y > 65535u) return NNIS_ERR_UNSUPPORTED;
         batched_linear_kernel<T><<<grid, 256, 0, stream>>>((const T*)A, lda, a_bs, (const T*)W,
-                                                           (T*)C, ldc, c_bs, M, N, K);
+                                                           (T*)C, ldc, c_bs, M, N, K, gate, gate_ld);
     }
     NNIS_RETURN_LAUNCH();
 }
@@ -128,13 +136,13 @@ static int launch_batched(const void* A, long long lda, long long a_bs, const vo
 }  // namespace nnis
 
 NNIS_API int nnis_batched_linear(const void* A, long long lda, long long a_bs, const void* W, void* C,
-                                 long long ldc, long long c_bs, int batch, int M, int N, int K,
-                                 int dtype, cudaStream_t stream) {
+                                 long long ldc, long long c_bs, int batch, int M, int N, int K, const float* gate,
+                                 long long gate_ld, int dtype, cudaStream_t stream) {
     if (!A || !W || !C || batch <= 0 || M <= 0 || N <= 0 || K <= 0 || batch > 65535)
         return NNIS_ERR_ARGUMENT;
     if (dtype == NNIS_DTYPE_F32)
-        return nnis::launch_batched<float>(A, lda, a_bs, W, C, ldc, c_bs, batch, M, N, K, stream);
+        return nnis::launch_batched<float>(A, lda, a_bs, W, C, ldc, c_bs, batch, M, N, K, gate, gate_ld, stream);
     if (dtype == NNIS_DTYPE_BF16)
-        return nnis::launch_batched<nnis::bf16>(A, lda, a_bs, W, C, ldc, c_bs, batch, M, N, K, stream);
+        return nnis::launch_batched<nnis::bf16>(A, lda, a_bs, W, C, ldc, c_bs, batch, M, N, K, gate, gate_ld, stream);
     return NNIS_ERR_UNSUPPORTED;
 }

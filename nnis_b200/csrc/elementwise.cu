@@ -125,11 +125,11 @@ rmsnorm_rows_kernel(const float* __restrict__ x, const int* __restrict__ rows,
 }
 
 // ---------------------------------------------------------------------------
-// out[n, i] = silu(g[n, i]) * u[n, i]; gate and up are the two halves of one
+// out[n, i] = act(g[n, i]) * u[n, i], act silu or gelu's tanh form; gate and up are the two halves of one
 // float32 row [2 * inter].  NNIS: crates/nnis-model/src/fused_swiglu.rs:14-27.
 // ---------------------------------------------------------------------------
-template <typename T>
-__global__ void silu_mul_kernel(const float* __restrict__ gate_up, T* __restrict__ out,
+template <typename T, bool GELU>
+__global__ void gate_mul_kernel(const float* __restrict__ gate_up, T* __restrict__ out,
                                 size_t n_rows, int inter) {
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= n_rows * (size_t)inter) return;
@@ -137,7 +137,9 @@ __global__ void silu_mul_kernel(const float* __restrict__ gate_up, T* __restrict
     int i = (int)(idx - n * inter);
     float g = gate_up[n * 2 * inter + i];
     float u = gate_up[n * 2 * inter + inter + i];
-    out[idx] = from_float<T>((g / (1.0f + expf(-g))) * u);
+    const float act = GELU ? 0.5f * g * (1.0f + tanhf(0.79788456080286536f * (g + 0.044715f * g * g * g)))
+                           : g / (1.0f + expf(-g));
+    out[idx] = from_float<T>(act * u);
 }
 
 // ---------------------------------------------------------------------------
@@ -362,9 +364,23 @@ NNIS_API int nnis_silu_mul(const float* gate_up, void* out, int out_dtype, long 
     size_t total = (size_t)n_rows * inter;
     unsigned blocks = (unsigned)((total + 255) / 256);
     if (out_dtype == NNIS_DTYPE_F32)
-        silu_mul_kernel<float><<<blocks, 256, 0, stream>>>(gate_up, (float*)out, n_rows, inter);
+        gate_mul_kernel<float, false><<<blocks, 256, 0, stream>>>(gate_up, (float*)out, n_rows, inter);
     else if (out_dtype == NNIS_DTYPE_BF16)
-        silu_mul_kernel<bf16><<<blocks, 256, 0, stream>>>(gate_up, (bf16*)out, n_rows, inter);
+        gate_mul_kernel<bf16, false><<<blocks, 256, 0, stream>>>(gate_up, (bf16*)out, n_rows, inter);
+    else
+        return NNIS_ERR_UNSUPPORTED;
+    NNIS_RETURN_LAUNCH();
+}
+
+NNIS_API int nnis_gelu_mul(const float* gate_up, void* out, int out_dtype, long long n_rows, int inter,
+                           cudaStream_t stream) {
+    if (n_rows <= 0 || inter <= 0) return NNIS_ERR_ARGUMENT;
+    size_t total = (size_t)n_rows * inter;
+    unsigned blocks = (unsigned)((total + 255) / 256);
+    if (out_dtype == NNIS_DTYPE_F32)
+        gate_mul_kernel<float, true><<<blocks, 256, 0, stream>>>(gate_up, (float*)out, n_rows, inter);
+    else if (out_dtype == NNIS_DTYPE_BF16)
+        gate_mul_kernel<bf16, true><<<blocks, 256, 0, stream>>>(gate_up, (bf16*)out, n_rows, inter);
     else
         return NNIS_ERR_UNSUPPORTED;
     NNIS_RETURN_LAUNCH();

@@ -66,7 +66,7 @@ struct GemmArgs {
     // (it is read ahead of this kernel's wait, with the first loads of W).
     const int* tile_expert;
     int expert_rows;
-    // an activation in the storing epilogues: 0 none; 1 relu(x)^2 (the experts'); 2 gelu with erf,
+    // an activation in the storing epilogues (3 in the gated one too, in silu's place): 0 none; 1 relu(x)^2 (the experts'); 2 gelu with erf,
     // 0.5 x (1 + erf(x / sqrt 2)); 3 gelu's tanh form
     int act;
     // GEMM_GATED with glu_limit > 0: the clamped form g' sigmoid(glu_alpha g') (u' + 1) with
@@ -457,7 +457,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
                             uv = fminf(fmaxf(uv, -g.glu_limit), g.glu_limit) + 1.0f;
                             slope *= g.glu_alpha;
                         }
-                        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(gv * slope));
+                        float arg = gv * slope;
+                        // gelu's tanh form is z sigmoid(2 sqrt(2 / pi) (z + 0.044715 z^3))
+                        if (g.act == GEMM_ACT_GELU_TANH)
+                            arg *= 1.5957691216057308f * fmaf(0.044715f * gv, gv, 1.0f);
+                        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(arg));
                         asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
                         f[i] = gv * r * uv;
                     }
@@ -618,7 +622,9 @@ static int gemm_tc_run(const void* A, const void* W, const float* bias, void* C,
                        cudaStream_t stream, float glu_limit, float glu_alpha, int act = 0) {
     using namespace nnis;
     if (M <= 0 || N <= 0 || K <= 0 || !A || !W || !C || mode < 0 || mode > 4) return NNIS_ERR_ARGUMENT;
-    if (act < 0 || act > GEMM_ACT_GELU_TANH || (act && mode != GEMM_STORE)) return NNIS_ERR_ARGUMENT;
+    if (act < 0 || act > GEMM_ACT_GELU_TANH) return NNIS_ERR_ARGUMENT;
+    if (act && mode != GEMM_STORE && !(mode == GEMM_GATED && act == GEMM_ACT_GELU_TANH && !(glu_limit > 0.f)))
+        return NNIS_ERR_ARGUMENT;
     if (K % 8) return NNIS_ERR_UNSUPPORTED;
     if (((uintptr_t)A | (uintptr_t)W) % 16) return NNIS_ERR_ALIGNMENT;
     if (((uintptr_t)C % 16) != 0) return NNIS_ERR_ALIGNMENT;
@@ -715,6 +721,14 @@ NNIS_API int nnis_gemm_tc_glu_clamp(const void* A, const void* W, const float* b
     if (!(limit > 0.f)) return NNIS_ERR_ARGUMENT;
     return gemm_tc_run(A, W, bias, C, M, N, K, 3, nullptr, nullptr, nullptr, 0, nullptr, nullptr, nullptr, nullptr,
                        0, 0, 0, 0, nullptr, 0, nullptr, 0, sm_count, status, pdl, stream, limit, alpha);
+}
+
+// The gated product (mode 3) with gelu's tanh form in its epilogue: out [M, N / 2] = bf16(gelu(gate) * up).
+NNIS_API int nnis_gemm_tc_gelu_gated(const void* A, const void* W, const float* bias, void* C, int M, int N, int K,
+                                     int sm_count, int* status, int pdl, cudaStream_t stream) {
+    return gemm_tc_run(A, W, bias, C, M, N, K, 3, nullptr, nullptr, nullptr, 0, nullptr, nullptr, nullptr, nullptr,
+                       0, 0, 0, 0, nullptr, 0, nullptr, 0, sm_count, status, pdl, stream, 0.f, 0.f,
+                       nnis::GEMM_ACT_GELU_TANH);
 }
 
 // The storing product (mode 0) with an activation in its epilogue: out [M, N] = bf16(act(A . W^T + bias)),

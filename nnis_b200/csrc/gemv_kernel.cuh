@@ -88,7 +88,8 @@ struct GemvArgs {
     const float* ss_parts;
     int ss_units;
     // STORE epilogue, optional: an activation on the sums before they are rounded; 0 none, 1 the square of
-    // relu, 2 gelu with erf, 3 gelu's tanh form (the codes of the tensor-core product's storing epilogue)
+    // relu, 2 gelu with erf, 3 gelu's tanh form (the codes of the tensor-core product's storing epilogue);
+    // GATED epilogue: the same on the gate's sums, in place of silu
     int act;
 };
 
@@ -291,9 +292,10 @@ __device__ __forceinline__ void epi_finish(const GemvArgs& a, int unit, int row0
                 vb[e] = pv[hrow * 2 + e] + bias_b[e];
             }
             if (EPI == EPI_GATED) {
+                const float g0 = a.act ? gemv_act(va[0], a.act) : va[0] / (1.0f + expf(-va[0]));
+                const float g1 = a.act ? gemv_act(va[1], a.act) : va[1] / (1.0f + expf(-va[1]));
                 *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(a.out) + (size_t)m * inter + n_a) =
-                    pack_bf16((va[0] / (1.0f + expf(-va[0]))) * vb[0],
-                              (va[1] / (1.0f + expf(-va[1]))) * vb[1]);
+                    pack_bf16(g0 * vb[0], g1 * vb[1]);
             } else {
                 int pos = p.pos[hrow];
                 if (pos < 0) continue;

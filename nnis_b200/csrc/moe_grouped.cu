@@ -88,7 +88,8 @@ __global__ void __launch_bounds__(128)
 grouped_mma_kernel(const bf16* __restrict__ a, int lda, const int* __restrict__ perm, int top,
                    const bf16* __restrict__ w, const int* __restrict__ tile_expert,
                    void* __restrict__ out, int N, int K, int M, long long a_bs, int ldc,
-                   long long c_bs, const float* __restrict__ pair_weight = nullptr, int act = 1) {
+                   long long c_bs, const float* __restrict__ pair_weight = nullptr, int act = 1,
+                   const float* __restrict__ gate = nullptr, long long gate_ld = 0) {
     constexpr int BK = 64, STAGES = 3, CH = BK / 8;
     const int expert = MODE == 2 ? (int)blockIdx.z : tile_expert[blockIdx.x];
     if (expert < 0) return;
@@ -167,6 +168,11 @@ grouped_mma_kernel(const bf16* __restrict__ a, int lda, const int* __restrict__ 
             float v0 = acc[j][h * 2], v1 = acc[j][h * 2 + 1];
             if (MODE == 2) {
                 bf16* o = reinterpret_cast<bf16*>(out);
+                if (gate) {  // the sigmoid of a logit per output value
+                    const float* z = gate + (size_t)(row0 + r) * gate_ld + (size_t)expert * N + col;
+                    if (col < N) v0 *= 1.0f / (1.0f + expf(-z[0]));
+                    if (col + 1 < N) v1 *= 1.0f / (1.0f + expf(-z[1]));
+                }
                 if (col < N) o[base + col] = __float2bfloat16_rn(v0);
                 if (col + 1 < N) o[base + col + 1] = __float2bfloat16_rn(v1);
             } else if (MODE == 3) {  // (v0, v1) = (gate, up) of feature col / 2; the score on both
@@ -271,11 +277,12 @@ static int configure_grouped() {
 }
 
 // One matrix per head on packed bfloat16 rows, on the tensor cores (what nnis_batched_linear
-// computes on the CUDA cores): out[m, b * c_bs : + N] = a[m, b * a_bs : + K] . w[b]^T.  Takes
+// computes on the CUDA cores): out[m, b * c_bs : + N] = a[m, b * a_bs : + K] . w[b]^T, times the sigmoid of
+// gate[m, b * N : + N] if gate is given.  Takes
 // K, lda, a_bs in multiples of 8 and 16-byte aligned a and w; else NNIS_ERR_UNSUPPORTED.
 NNIS_API int nnis_batched_linear_mma(const void* a, long long lda, long long a_bs, const void* w, void* out,
                                      long long ldc, long long c_bs, int batch, int M, int N, int K,
-                                     cudaStream_t stream) {
+                                     const float* gate, long long gate_ld, cudaStream_t stream) {
     if (!a || !w || !out || batch <= 0 || M <= 0 || N <= 0 || K <= 0) return NNIS_ERR_ARGUMENT;
     if (K % 8 || lda % 8 || a_bs % 8 || ((uintptr_t)a | (uintptr_t)w) % 16 || batch > 65535 ||
         lda > 0x7fffffff || ldc > 0x7fffffff)
@@ -286,7 +293,7 @@ NNIS_API int nnis_batched_linear_mma(const void* a, long long lda, long long a_b
     if (grid.y > 65535u) return NNIS_ERR_UNSUPPORTED;
     grouped_mma_kernel<2><<<grid, 128, kGroupedSmem, stream>>>((const bf16*)a, (int)lda, nullptr, 1,
                                                                (const bf16*)w, nullptr, out, N, K, M, a_bs,
-                                                               (int)ldc, c_bs);
+                                                               (int)ldc, c_bs, nullptr, 1, gate, gate_ld);
     NNIS_RETURN_LAUNCH();
 }
 

@@ -136,6 +136,16 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
                                 ctypes.c_longlong(n), inter, _stream()), "silu_mul")
 
 
+def gelu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
+    """out = gelu(gate_up[:, :I]) * gate_up[:, I:] with gelu's tanh form, gate_up float32 [n, 2I]."""
+    _cuda(gate_up, out)
+    n, inter = out.shape
+    _need(gate_up.dtype == torch.float32 and tuple(gate_up.shape) == (n, 2 * inter),
+          "gate_up: float32 [n, 2 * inter]")
+    _check(_lib().nnis_gelu_mul(_ptr(gate_up), _ptr(out), code_of(out.dtype),
+                                ctypes.c_longlong(n), inter, _stream()), "gelu_mul")
+
+
 def rope_store(qkv: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
                page_table: Optional[torch.Tensor], cos: Optional[torch.Tensor],
                sin: Optional[torch.Tensor], k_cache: Optional[torch.Tensor],
@@ -363,7 +373,8 @@ def gemv_bf16(w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, 
     times ``norm_weight`` (float32 [n]), to ``x_next`` (bfloat16 [m, n]) and every eight
     columns' sum of squares to ``shares`` (float32 [m, n / 8]).  The projection after it
     takes ``x=x_next, shares=shares, eps=`` the norm's, and scales its sums by
-    ``1 / sqrt(mean of squares + eps)`` (``gemv_shares_norm`` says whether it can)."""
+    ``1 / sqrt(mean of squares + eps)`` (``gemv_shares_norm`` says whether it can).
+    ``act``: an activation of the sums (EPI_STORE) or of the gate's sums in silu's place (EPI_GATED)."""
     _cuda(w, bias, out, x, hidden, norm_weight, rows, token_pos, token_seq, page_table, cos, sin,
           k_cache, v_cache, logits, scratch, next_tokens, next_pos, shares, *(emit or ()))
     n, k = w.shape
@@ -399,8 +410,9 @@ def gemv_bf16(w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, 
               "gemv: emit shares float32 [m, n / 8]")
     if bias is not None:
         _need(bias.dtype == torch.float32 and bias.numel() == n, "gemv: bias float32 [n]")
-    _need(act == 0 or (epilogue == EPI_STORE and act in (GEMM_ACT_RELU2, GEMM_ACT_GELU_ERF, GEMM_ACT_GELU_TANH)),
-          "gemv: an activation goes with the storing epilogue")
+    _need(act == 0 or (epilogue in (EPI_STORE, EPI_GATED)
+                       and act in (GEMM_ACT_RELU2, GEMM_ACT_GELU_ERF, GEMM_ACT_GELU_TANH)),
+          "gemv: an activation goes with the storing or the gated epilogue")
     if epilogue == EPI_STORE:
         _need(out.dtype == torch.bfloat16 and tuple(out.shape) == (m, n), "gemv: out bfloat16 [m, n]")
     elif epilogue in (EPI_STORE_F32, EPI_ADD_F32):
@@ -893,6 +905,22 @@ def gemm_tc_glu_clamp(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Ten
                                          PDL, _stream()), "gemm_tc_glu_clamp")
 
 
+def gemm_tc_gelu_gated(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """The gated tensor-core product with gelu's tanh form in its epilogue: w = [gate; up] rows, out
+    bfloat16 [m, n / 2] = gelu(gate) * up."""
+    _cuda(a, w, bias, out)
+    m, k = a.shape
+    n = w.shape[0]
+    _need(a.dtype == w.dtype == torch.bfloat16 and w.shape[1] == k, "gemm_tc_gelu_gated: bfloat16 a [m, k], w [n, k]")
+    _need(gemm_tc_takes(m, n, k), f"gemm_tc_gelu_gated: shape m={m} n={n} k={k} is not taken")
+    _need(n % 2 == 0 and out.dtype == torch.bfloat16 and tuple(out.shape) == (m, n // 2),
+          "gemm_tc_gelu_gated: out bfloat16 [m, n / 2]")
+    if bias is not None:
+        _need(bias.dtype == torch.float32 and bias.numel() == n, "gemm_tc_gelu_gated: bias float32 [n]")
+    _check(_lib().nnis_gemm_tc_gelu_gated(_ptr(a), _ptr(w), _ptr(bias), _ptr(out), m, n, k, sm_count(a.device),
+                                          _ptr(status_word(a.device)), PDL, _stream()), "gemm_tc_gelu_gated")
+
+
 def gemm_tc_act(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor, act: int) -> None:
     """The storing tensor-core product with an activation in its epilogue: out bfloat16 [m, n] =
     act(a . w^T + bias); ``GEMM_ACT_RELU2``, ``GEMM_ACT_GELU_ERF`` or ``GEMM_ACT_GELU_TANH``."""
@@ -1030,12 +1058,20 @@ def rope_part(src: torch.Tensor, src_head: int, src_off: int, dst: torch.Tensor,
            "rope_part")
 
 
-def batched_linear(a: torch.Tensor, a_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int) -> None:
+def batched_linear(a: torch.Tensor, a_head: int, w: torch.Tensor, out: torch.Tensor, out_head: int,
+                   gate: Optional[torch.Tensor] = None, gate_off: int = 0) -> None:
     """out[m, b * out_head : + N] = a[m, b * a_head : + K] . w[b]^T for every head b;
-    w [heads, N, K]; a and out packed rows whose heads are ``a_head`` / ``out_head`` apart."""
-    _cuda(a, w, out)
+    w [heads, N, K]; a and out packed rows whose heads are ``a_head`` / ``out_head`` apart.  ``gate``
+    (float32 rows with one logit per output value from column ``gate_off`` on): a sum is multiplied by
+    the sigmoid of its logit before it is rounded."""
+    _cuda(a, w, out, gate)
     heads, n, k = w.shape
     m = a.shape[0]
+    gate_ptr, gate_ld = ctypes.c_void_p(0), 0
+    if gate is not None:
+        _need(gate.dtype == torch.float32 and gate.dim() == 2 and gate.shape[0] == m
+              and 0 <= gate_off and gate_off + heads * n <= gate.shape[1], "batched_linear: gate float32 [m, >= heads * N]")
+        gate_ptr, gate_ld = ctypes.c_void_p(gate.data_ptr() + 4 * gate_off), gate.shape[1]
     _need(a.dtype == w.dtype == out.dtype and out.shape[0] == m, "batched_linear: one dtype, equal rows")
     _need(k <= a_head and (heads - 1) * a_head + k <= a.shape[1], "batched_linear: K lies outside a's heads")
     _need(n <= out_head and (heads - 1) * out_head + n <= out.shape[1],
@@ -1045,13 +1081,13 @@ def batched_linear(a: torch.Tensor, a_head: int, w: torch.Tensor, out: torch.Ten
         # many rows: 64 x 64 tiles on the tensor cores (the grouped products' kernel)
         _check(_lib().nnis_batched_linear_mma(_ptr(a), ctypes.c_longlong(a.shape[1]), ctypes.c_longlong(a_head),
                                               _ptr(w), _ptr(out), ctypes.c_longlong(out.shape[1]),
-                                              ctypes.c_longlong(out_head), heads, m, n, k, _stream()),
-               "batched_linear_mma")
+                                              ctypes.c_longlong(out_head), heads, m, n, k, gate_ptr,
+                                              ctypes.c_longlong(gate_ld), _stream()), "batched_linear_mma")
         return
     _check(_lib().nnis_batched_linear(_ptr(a), ctypes.c_longlong(a.shape[1]), ctypes.c_longlong(a_head),
                                       _ptr(w), _ptr(out), ctypes.c_longlong(out.shape[1]),
-                                      ctypes.c_longlong(out_head), heads, m, n, k, code_of(a.dtype),
-                                      _stream()), "batched_linear")
+                                      ctypes.c_longlong(out_head), heads, m, n, k, gate_ptr,
+                                      ctypes.c_longlong(gate_ld), code_of(a.dtype), _stream()), "batched_linear")
 
 
 def latent_prep(a: torch.Tensor, wq: torch.Tensor, wkv: torch.Tensor, freq: torch.Tensor,
@@ -1080,11 +1116,12 @@ def latent_prep(a: torch.Tensor, wq: torch.Tensor, wkv: torch.Tensor, freq: torc
 def latent_prep_direct(a: torch.Tensor, wkv: torch.Tensor, freq: torch.Tensor, token_pos: torch.Tensor,
                        token_seq: torch.Tensor, page_table: torch.Tensor, q_plain: torch.Tensor,
                        q_rows: torch.Tensor, cache: torch.Tensor, gate: Optional[torch.Tensor], heads: int, dim: int,
-                       kv_rank: int, rot: int, rot_dims: int, eps: float, pairing: str = "half") -> None:
+                       kv_rank: int, rot: int, rot_dims: int, eps: float, pairing: str = "half", magnitude: float = 1.0) -> None:
     """From float32 rows [q (heads x (dim plain | rot rotated)) | c raw | kr raw | gate logits]: the plain
     parts of q packed to ``q_plain`` [n, heads * dim], the rotated ones turned into the last ``rot``
     values of every head of ``q_rows`` [n, heads * (kv_rank + rot)], the normed c and the turned kr
-    into the cache row of each token, and the sigmoid of the gate's logits (``gate`` [n, heads] or None)."""
+    into the cache row of each token, and the sigmoid of the gate's logits (``gate`` [n, heads] or None).
+    ``magnitude`` multiplies every cosine and sine."""
     _cuda(a, wkv, freq, token_pos, token_seq, page_table, q_plain, q_rows, cache, gate)
     n = a.shape[0]
     _need(pairing in ("neighbours", "half"), "latent_prep_direct: pairing is neighbours or half")
@@ -1103,19 +1140,21 @@ def latent_prep_direct(a: torch.Tensor, wkv: torch.Tensor, freq: torch.Tensor, t
                                           _ptr(page_table), page_table.shape[1], _ptr(q_plain), _ptr(q_rows),
                                           _ptr(cache), _ptr(gate), n, heads, dim, kv_rank, rot, rot_dims,
                                           cache.shape[2], ctypes.c_float(eps), 1 if pairing == "neighbours" else 0,
-                                          a.shape[1], code_of(q_plain.dtype), _stream()), "latent_prep_direct")
+                                          a.shape[1], ctypes.c_float(magnitude), code_of(q_plain.dtype), _stream()),
+           "latent_prep_direct")
 
 
 def attention_latent(q: torch.Tensor, cache: torch.Tensor, token_pos: torch.Tensor,
                      token_seq: torch.Tensor, page_table: torch.Tensor, out: torch.Tensor, heads: int,
                      dv: int, scale: float, n_splits: int = 1,
                      partial: Optional[torch.Tensor] = None, window: int = 0,
-                     gate: Optional[torch.Tensor] = None) -> None:
+                     gate: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> None:
     """Causal attention of packed queries [n, heads * dk] over cache rows [pages, 1, page,
     dk] shared by all heads; the rows' first ``dv`` values are the values.  out [n, heads * dv].
     ``window`` > 0: a query sees that many keys, itself included; ``gate`` (float32 [n, heads])
-    multiplies each head's output."""
-    _cuda(q, cache, token_pos, token_seq, page_table, out, partial, gate)
+    multiplies each head's output; ``sink`` (float32 [heads]): the denominator also holds exp(sink)."""
+    _cuda(q, cache, token_pos, token_seq, page_table, out, partial, gate, sink)
+    _need(sink is None or (sink.dtype == torch.float32 and sink.numel() == heads), "attention_latent: sink [heads]")
     _need(gate is None or (gate.dtype == torch.float32 and gate.numel() >= out.shape[0] * heads), "attention_latent: gate")
     n = out.shape[0]
     pages, one, page_size, dk = cache.shape
@@ -1129,7 +1168,7 @@ def attention_latent(q: torch.Tensor, cache: torch.Tensor, token_pos: torch.Tens
     _check(_lib().nnis_attention_latent(_ptr(q), _ptr(cache), _ptr(token_pos), _ptr(token_seq),
                                         _ptr(page_table), page_table.shape[1], _ptr(out), _ptr(partial), n,
                                         heads, dk, dv, page_size, ctypes.c_float(scale), n_splits, window,
-                                        _ptr(gate), code_of(out.dtype), _stream()),
+                                        _ptr(gate), _ptr(sink), code_of(out.dtype), _stream()),
            "attention_latent", 2 if n_splits > 1 else 1)
 
 
@@ -1267,12 +1306,13 @@ def attention_latent_mma(q: torch.Tensor, cache: torch.Tensor, tiles: Optional[t
                          seq_count: Optional[torch.Tensor], token_pos: torch.Tensor, token_seq: torch.Tensor,
                          page_table: torch.Tensor, out: torch.Tensor, heads: int, dv: int, scale: float,
                          n_splits: int = 1, partial: Optional[torch.Tensor] = None, window: int = 0,
-                         gate: Optional[torch.Tensor] = None) -> None:
+                         gate: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> None:
     """``attention_latent`` on the tensor cores (bfloat16).  With ``tiles`` (``latent_tiles``) a
     prompt step; without, every row is one token of a sequence of its own."""
-    _cuda(q, cache, tiles, seq_first_row, seq_start, seq_count, token_pos, token_seq, page_table, out, partial, gate)
+    _cuda(q, cache, tiles, seq_first_row, seq_start, seq_count, token_pos, token_seq, page_table, out, partial, gate, sink)
     n = out.shape[0]
     _need(gate is None or (gate.dtype == torch.float32 and gate.numel() >= n * heads), "attention_latent_mma: gate")
+    _need(sink is None or (sink.dtype == torch.float32 and sink.numel() == heads), "attention_latent_mma: sink [heads]")
     pages, one, page_size, dk = cache.shape
     _need(q.dtype == cache.dtype == out.dtype == torch.bfloat16, "attention_latent_mma: bfloat16")
     _need(one == 1 and q.shape[1] == heads * dk and out.shape[1] == heads * dv, "attention_latent_mma: shapes")
@@ -1285,7 +1325,7 @@ def attention_latent_mma(q: torch.Tensor, cache: torch.Tensor, tiles: Optional[t
         _ptr(q), _ptr(cache), _ptr(tiles), tiles.shape[0] if tiles is not None else 0, _ptr(seq_first_row),
         _ptr(seq_start), _ptr(seq_count), _ptr(token_pos), _ptr(token_seq), _ptr(page_table),
         page_table.shape[1], _ptr(out), _ptr(partial), n, heads, dk, dv, page_size, ctypes.c_float(scale),
-        n_splits, window, _ptr(gate), _stream()), "attention_latent_mma", 2 if n_splits > 1 else 1)
+        n_splits, window, _ptr(gate), _ptr(sink), _stream()), "attention_latent_mma", 2 if n_splits > 1 else 1)
 
 
 
@@ -1590,7 +1630,7 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
              v_cache: Optional[torch.Tensor], gate_out: Optional[torch.Tensor], heads: int, kv_heads: int,
              dk: int, dv: int, rot: int, eps: float, pairing: str = "neighbours", head_norm: bool = False,
              q_scale: Optional[torch.Tensor] = None, maps: int = 1, magnitude: float = 1.0,
-             head_weights=None) -> None:
+             head_weights=None, values_are_keys: bool = False) -> None:
     """From float32 rows [q | k | v | gate logits]: norms of q and k, rotation, q packed, k and v into
     the cache, sigmoid of the gate's logits (``gate_out`` [n, heads] or [n, heads * dv]: as many logits a
     row).  ``kv_heads == 0``: the rows hold no keys and values.  Two forms: with ``wq``/``wk`` the
@@ -1600,7 +1640,8 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
     every head divided by its own root mean square.  ``maps`` > 1: a head of q or k holds that many
     vectors of dk / maps values side by side, each turned by itself over its first ``rot`` values;
     ``magnitude`` multiplies every cosine and sine.  ``head_weights``: (q's, k's), float32 [dk] each or
-    None: every head of q (k) normed by itself with that weight, before the rotation (the per-head form)."""
+    None: every head of q (k) normed by itself with that weight, before the rotation (the per-head form).
+    ``values_are_keys`` (per-head form): the rows hold no v; the values are the keys as projected."""
     hq, hk = head_weights if head_weights is not None else (None, None)
     _cuda(hq, hk)
     for w in (hq, hk):
@@ -1609,7 +1650,9 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
     n = a.shape[0]
     gate_cols = 0 if gate_out is None else gate_out.shape[1]
     _need(gate_cols in (0, heads, heads * dv), "qkv_prep: a gate per head or per value")
-    _need(a.dtype == torch.float32 and a.shape[1] == heads * dk + kv_heads * (dk + dv) + gate_cols,
+    _need(not values_are_keys or dk == dv, "qkv_prep: values that are the keys have their size")
+    _need(a.dtype == torch.float32
+          and a.shape[1] == heads * dk + kv_heads * (dk + (0 if values_are_keys else dv)) + gate_cols,
           "qkv_prep: float32 rows [q | k | v | gate]")
     _need(tuple(q_out.shape) == (n, heads * dk), "qkv_prep: q_out [n, heads * dk]")
     for w, size in ((wq, heads * dk), (wk, kv_heads * dk)):
@@ -1625,7 +1668,7 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
         _need(page_table is not None and page_table.dtype == torch.int32, "qkv_prep: page_table int32")
         cols, page_size = page_table.shape[1], k_cache.shape[2]
     per_head = head_norm or pairing == "half" or q_scale is not None or gate_cols not in (0, heads) \
-        or maps != 1 or magnitude != 1.0 or head_weights is not None
+        or maps != 1 or magnitude != 1.0 or head_weights is not None or values_are_keys
     _need(maps >= 1 and dk % maps == 0 and rot <= dk // maps, "qkv_prep: maps vectors of equal size in a head")
     if per_head:
         _need(wq is None and wk is None, "qkv_prep: the per-head form has no norm over the whole projections")
@@ -1636,7 +1679,7 @@ def qkv_prep(a: torch.Tensor, wq: Optional[torch.Tensor], wk: Optional[torch.Ten
                                           _ptr(gate_out), n, heads, kv_heads, dk, dv, rot,
                                           1 if pairing == "half" else 0, 1 if head_norm else 0, gate_cols,
                                           page_size, ctypes.c_float(eps), maps, ctypes.c_float(magnitude),
-                                          code_of(q_out.dtype), _stream()),
+                                          1 if values_are_keys else 0, code_of(q_out.dtype), _stream()),
                "qkv_prep_heads")
         return
     _check(_lib().nnis_qkv_prep(_ptr(a), _ptr(wq), _ptr(wk), _ptr(freq), _ptr(token_pos), _ptr(token_seq),
@@ -2065,3 +2108,77 @@ def attention_diff_mma(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Te
                                           page_table.shape[1], _ptr(gate), _ptr(out), heads, kv_heads, dk2 // 2, dv,
                                           page_size, window, ctypes.c_float(scale), ctypes.c_float(lam),
                                           ctypes.c_float(post), ctypes.c_float(eps), _stream()), "attention_diff_mma")
+
+
+# ---- matrix memory (csrc/matrix_memory.cu) --------------------------------------------------
+def memory_chunk_tokens() -> int:
+    """Tokens of a chunk of a prompt step's matrix memory."""
+    return int(_lib().nnis_memory_chunk_tokens())
+
+
+def _memory_args(a, i_bias, f_bias, state, norm_state, max_state, o_raw, heads, dim, vdim):
+    n = a.shape[0]
+    _need(a.dtype == torch.float32 and a.dim() == 2 and a.shape[1] >= 2 * heads * (dim + vdim) + 2 * heads,
+          "matrix memory: float32 rows [q | k | v | g | i | f]")
+    for t in (i_bias, f_bias):
+        _need(t.dtype == torch.float32 and t.numel() == heads, "matrix memory: gate biases float32 [heads]")
+    slots = state.shape[0]
+    _need(state.dtype == norm_state.dtype == max_state.dtype == torch.float32
+          and tuple(state.shape) == (slots, heads, dim, vdim) and tuple(norm_state.shape) == (slots, 2, heads, dim)
+          and tuple(max_state.shape) == (slots, 2, heads), "matrix memory: state shapes")
+    _need(o_raw.dtype == torch.float32 and tuple(o_raw.shape) == (n, heads * vdim), "matrix memory: o [n, heads * vdim]")
+
+
+def memory_step(a: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, state: torch.Tensor,
+                norm_state: torch.Tensor, max_state: torch.Tensor, token_pos: torch.Tensor, token_seq: torch.Tensor,
+                seq_slots: torch.Tensor, o_raw: torch.Tensor, heads: int, dim: int, vdim: int, cap: float,
+                q_scale: float, floor: float) -> None:
+    """One token per row: the matrix memory of every row's slot moved on by its token, and the token's
+    output before the head norm.  The normaliser and the running maximum are kept twice: position p
+    reads number p & 1 and leaves the other."""
+    _cuda(a, i_bias, f_bias, state, norm_state, max_state, token_pos, token_seq, seq_slots, o_raw)
+    _memory_args(a, i_bias, f_bias, state, norm_state, max_state, o_raw, heads, dim, vdim)
+    _check(_lib().nnis_memory_step(_ptr(a), a.shape[1], _ptr(i_bias), _ptr(f_bias), _ptr(state), _ptr(norm_state),
+                                   _ptr(max_state), _ptr(token_pos), _ptr(token_seq), _ptr(seq_slots), _ptr(o_raw),
+                                   a.shape[0], heads, dim, vdim, ctypes.c_float(cap), ctypes.c_float(q_scale),
+                                   ctypes.c_float(floor), _stream()), "memory_step")
+
+
+def memory_prompt(a: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, state: torch.Tensor,
+                  norm_state: torch.Tensor, max_state: torch.Tensor, chunks: torch.Tensor,
+                  seq_first_chunk: torch.Tensor, seq_slots: torch.Tensor, seq_first_row: torch.Tensor,
+                  seq_start: torch.Tensor, seq_count: torch.Tensor, gates: torch.Tensor, chunk_gates: torch.Tensor,
+                  chunk_state: torch.Tensor, chunk_norm: torch.Tensor, o_raw: torch.Tensor, heads: int, dim: int,
+                  vdim: int, cap: float, q_scale: float, floor: float) -> None:
+    """``memory_step`` for prompt steps, chunk by chunk (``scan_segments`` of ``memory_chunk_tokens``).  Scratch:
+    ``gates`` float64 [3, n, heads], ``chunk_gates`` float64 [3, chunks, heads], ``chunk_state`` float32
+    [chunks, heads, dim, vdim], ``chunk_norm`` float32 [chunks, heads, dim]."""
+    _cuda(a, i_bias, f_bias, state, norm_state, max_state, chunks, seq_first_chunk, seq_slots, seq_first_row, seq_start,
+          seq_count, gates, chunk_gates, chunk_state, chunk_norm, o_raw)
+    _memory_args(a, i_bias, f_bias, state, norm_state, max_state, o_raw, heads, dim, vdim)
+    n, c, seqs = a.shape[0], chunks.shape[0], seq_count.numel()
+    _need(chunks.dtype == torch.int32 and chunks.dim() == 2 and chunks.shape[1] == 2
+          and seq_first_chunk.dtype == torch.int32 and seq_first_chunk.numel() == seqs + 1, "memory_prompt: chunk lists")
+    _need(gates.dtype == chunk_gates.dtype == torch.float64 and gates.numel() >= 3 * n * heads
+          and chunk_gates.numel() >= 3 * c * heads, "memory_prompt: float64 gate scratch")
+    _need(chunk_state.dtype == chunk_norm.dtype == torch.float32 and chunk_state.numel() >= c * heads * dim * vdim
+          and chunk_norm.numel() >= c * heads * dim, "memory_prompt: chunk scratch")
+    _check(_lib().nnis_memory_prompt(_ptr(a), a.shape[1], _ptr(i_bias), _ptr(f_bias), _ptr(state), _ptr(norm_state),
+                                     _ptr(max_state), _ptr(chunks), c, _ptr(seq_first_chunk), seqs, _ptr(seq_slots),
+                                     _ptr(seq_first_row), _ptr(seq_start), _ptr(seq_count), _ptr(gates),
+                                     _ptr(chunk_gates), _ptr(chunk_state), _ptr(chunk_norm), _ptr(o_raw), n, heads, dim,
+                                     vdim, ctypes.c_float(cap), ctypes.c_float(q_scale), ctypes.c_float(floor),
+                                     _stream()), "memory_prompt", 4)
+
+
+def memory_finish(o_raw: torch.Tensor, a: torch.Tensor, gate_off: int, weight: torch.Tensor, token_pos: torch.Tensor,
+                  out: torch.Tensor, heads: int, vdim: int, eps: float) -> None:
+    """out = o / rms(o) per head * weight * sigmoid(g), g the float32 columns of ``a`` from ``gate_off`` on."""
+    _cuda(o_raw, a, weight, token_pos, out)
+    n = o_raw.shape[0]
+    _need(o_raw.dtype == a.dtype == weight.dtype == torch.float32 and tuple(o_raw.shape) == (n, heads * vdim)
+          and tuple(out.shape) == (n, heads * vdim) and weight.numel() == heads * vdim
+          and a.shape[0] == n and gate_off + heads * vdim <= a.shape[1], "memory_finish: shapes")
+    _check(_lib().nnis_memory_finish(_ptr(o_raw), _ptr(a), a.shape[1], gate_off, _ptr(weight), _ptr(token_pos),
+                                     _ptr(out), n, heads, vdim, ctypes.c_float(eps), code_of(out.dtype), _stream()),
+           "memory_finish")

@@ -1,5 +1,5 @@
-from . import (attention, block, delta_rule, diff_attention, embedding, latent_attention, mixer_pair, mlp, moe,  # noqa: F401
-               norm, position, retention, selective_scan, sink_attention, wkv)  # (registration)
+from . import (attention, block, delta_rule, diff_attention, embedding, latent_attention, matrix_memory,  # noqa: F401
+               mixer_pair, mlp, moe, norm, position, retention, selective_scan, sink_attention, wkv)  # (registration)
 from .base import (BLOCKS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, POSITIONS, Part,
                    PositionEncoding, Registry)
 from .block import Block

@@ -284,7 +284,8 @@ class SandwichBlock(Block):
     x += norm2b(ffn(norm2(x))).  The sub-layer adds its output up in a zeroed float32 branch buffer,
     as it would into the residual stream, and one kernel norms that buffer and adds it to the stream
     (leaving the buffer zero again).  Roles: mixer_norm, mixer, mixer_post_norm and, optionally, ffn_norm,
-    ffn, ffn_post_norm; the norms after the sub-layers are RMS norms (``rmsnorm``).
+    ffn, ffn_post_norm; the norms after the sub-layers are RMS norms (``rmsnorm``).  ``LayerSpec.params["tolerated"]``
+    names tensor stems that a folder may hold although the layer has no use for them.
 
     ``LayerSpec.params["depth_mix"]`` = {"name": tensor stem, "terms": t, "most": m} turns on the depth-weighted
     average: with X_0 what the first such block of a run was given and X_t-1 this block's result, the
@@ -318,6 +319,9 @@ class SandwichBlock(Block):
 
     def weight_specs(self) -> Dict[str, WeightSpec]:
         specs = super().weight_specs()
+        # (a layer without a feed-forward has no use for its norms; a folder may still hold them)
+        for stem in self.spec.params.get("tolerated", ()):
+            specs.setdefault(f"{self.spec.prefix}.{stem}", WeightSpec((-1,), "unused"))
         if self.mix_name:
             specs[self.mix_name] = WeightSpec((self.mix_terms,), "vector", init="ones")
         return specs

@@ -12,7 +12,11 @@ With ``q_rank`` 0 there is no latent for the queries: ``q = W_q h``.  Then the q
 latent and, with ``gate`` "head", the logits of a gate per head (head i's output is multiplied
 by ``sigmoid(W_g h)_i``) come from one product of stacked matrices, and one kernel
 (``latent_prep_direct``) packs, turns, norms, stores and takes the sigmoid; the gate multiplies
-the weighted sum of latents, which is the head's output before its linear ``W_uv``.
+the weighted sum of latents, which is the head's output before its linear ``W_uv``.  With
+``gate`` "value" W_g has a row per output value and the joined heads are multiplied value by value
+by ``sigmoid(W_g h)``, in the epilogue of the product with ``W_uv``.  With ``sink`` the softmax's
+denominator also holds ``exp(sink_h)``, a learned number per head (names["sink"]) with no key and no
+value.  A position encoding with a ``magnitude`` multiplies every cosine and sine by it (q_rank 0).
 
 Only ``[c | k_rot]`` is cached, one row per position for all heads, in a cache
 group without storage for values.  Because ``q_plain . (W_uk c) = (W_uk^T q_plain) . c``,
@@ -22,9 +26,9 @@ product with the cached row, the output is a weighted sum of the rows' ``c`` par
 and the heads' values are made from that sum (``W_uv`` per head) before ``W_o`` adds
 into the residual stream.  Prompts, later chunks and single tokens take the same way.
 
-params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, eps, window, gate,
+params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, eps, window, gate, sink,
 position (a ``rope_frequencies`` PartSpec, either pairing), names {dq, dq_norm, uq (or q), dkv,
-dkv_norm, uk, uv, o, gate}.
+dkv_norm, uk, uv, o, gate, sink}.
 """
 from __future__ import annotations
 
@@ -53,9 +57,12 @@ class LatentAttention(Part):
         self.eps = float(params["eps"])
         self.window = int(params.get("window") or 0)
         gate = params.get("gate", False)
-        if gate not in (False, None, "head"):
-            raise ValueError(f"latent attention: gate {gate!r} is not known (head)")
+        if gate not in (False, None, "head", "value"):
+            raise ValueError(f"latent attention: gate {gate!r} is not known (head, value)")
         self.has_gate = bool(gate)
+        self.gate_by_value = gate == "value"
+        self.gate_cols = (self.heads * self.vdim if self.gate_by_value else self.heads) if self.has_gate else 0
+        self.has_sink = bool(params.get("sink", False))
         if self.has_gate and self.q_rank:
             raise ValueError("latent attention: a gate goes with queries straight from the input (q_rank 0)")
         self.names = params["names"]
@@ -66,6 +73,10 @@ class LatentAttention(Part):
         if self.position.dims > self.rot:
             raise ValueError(f"rotation over {self.position.dims} dimensions, the rotated part has {self.rot}")
         self.pairing = getattr(self.position, "pairing", "half")
+        self.magnitude = float(getattr(self.position, "magnitude", 1.0))
+        if self.magnitude != 1.0 and self.q_rank:
+            raise ValueError("latent attention: a rotation with a magnitude goes with queries straight from the input "
+                             "(q_rank 0)")
         for what in ("heads", "dim", "vdim", "kv_rank"):
             if getattr(self, what) <= 0:
                 raise ValueError(f"latent attention: {what} must be positive")
@@ -74,7 +85,7 @@ class LatentAttention(Part):
         self.row = self.kv_rank + self.rot  # a cached row, and a query in the latent's space
         self.q_cols = self.heads * (self.dim + self.rot)
         self.w_down = self.w_uq = self.w_ukt = self.w_uv = self.w_o = None
-        self.norm_q = self.norm_kv = None
+        self.norm_q = self.norm_kv = self.sink = None
 
     # -- weights ----------------------------------------------------------
     def _name(self, key: str) -> str:
@@ -91,7 +102,9 @@ class LatentAttention(Part):
         else:
             specs = {self._name("q"): WeightSpec((self.q_cols, W), "matrix", fan_in=W)}
         if self.has_gate:
-            specs[self._name("gate")] = WeightSpec((H, W), "matrix", fan_in=W)
+            specs[self._name("gate")] = WeightSpec((self.gate_cols, W), "matrix", fan_in=W)
+        if self.has_sink:
+            specs[self._name("sink")] = WeightSpec((H,), "vector")
         specs.update({
             self._name("dkv"): WeightSpec((self.kv_rank + self.rot, W), "matrix", fan_in=W),
             self._name("dkv_norm"): WeightSpec((self.kv_rank,), "vector", init="ones"),
@@ -113,6 +126,8 @@ class LatentAttention(Part):
             self.norm_q = tensors[self._name("dq_norm")]
             self.w_uq = tensors[self._name("uq")]
         self.norm_kv = tensors[self._name("dkv_norm")]
+        if self.has_sink:
+            self.sink = tensors[self._name("sink")]
         # per head [kv_rank, dim]: the product that carries q_plain into the latent's space
         self.w_ukt = tensors[self._name("uk")].view(H, self.dim, self.kv_rank).transpose(1, 2).contiguous()
         self.w_uv = tensors[self._name("uv")].view(H, self.vdim, self.kv_rank).contiguous()
@@ -133,7 +148,7 @@ class LatentAttention(Part):
     def step_flops(self, counts, starts) -> float:
         H, W = self.heads, self.hidden
         tokens = sum(counts)
-        into_q = W * self.q_rank + self.q_rank * self.q_cols if self.q_rank else W * (self.q_cols + (H if self.has_gate else 0))
+        into_q = W * self.q_rank + self.q_rank * self.q_cols if self.q_rank else W * (self.q_cols + self.gate_cols)
         per_token = into_q + W * self.row + H * self.dim * self.kv_rank + H * self.vdim * self.kv_rank + H * self.vdim * W
         keys = sum(sum(min(st + q + 1, self.window) for q in range(c)) if self.window
                    else c * st + c * (c + 1) // 2 for c, st in zip(counts, starts))
@@ -172,14 +187,15 @@ class LatentAttention(Part):
         down = ws.get("latent_down", (n, self.w_down.shape[0]), torch.float32)
         linear(x, self.w_down, None, down, STORE_F32, decode=ctx.decode)
         q_lat = ws.get("latent_q_abs", (n, H * self.row), self.dtype)
-        gate = ws.get("latent_gate", (n, H), torch.float32) if self.has_gate else None
+        # (a gate per head multiplies inside the attention kernel, one per value after W_uv)
+        gate = ws.get("latent_gate", (n, H), torch.float32) if self.has_gate and not self.gate_by_value else None
         if self.q_rank:
             self._queries_from_latent(ctx, down, q_lat, freq, table, cache)
         else:
             q = ws.get("latent_q", (n, H * self.dim), self.dtype)
             ops.latent_prep_direct(down, self.norm_kv, freq, ctx.token_pos, ctx.token_seq, table, q, q_lat, cache.k,
                                    gate, H, self.dim, self.kv_rank, self.rot, self.position.dims, self.eps,
-                                   pairing=self.pairing)
+                                   pairing=self.pairing, magnitude=self.magnitude)
             ops.batched_linear(q, self.dim, self.w_ukt, q_lat, self.row)
         o_lat = ws.get("latent_o", (n, H * self.kv_rank), self.dtype)
         tiles = ctx.tables.get(self._tiles_name())
@@ -190,11 +206,11 @@ class LatentAttention(Part):
             if ctx.decode:
                 ops.attention_latent_mma(q_lat, cache.k, None, None, None, None, ctx.token_pos, ctx.token_seq,
                                          table, o_lat, H, self.kv_rank, self.scale, splits, partial,
-                                         window=self.window, gate=gate)
+                                         window=self.window, gate=gate, sink=self.sink)
             else:
                 ops.attention_latent_mma(q_lat, cache.k, tiles, ctx.seq_first_row, ctx.seq_start,
                                          ctx.seq_count, ctx.token_pos, ctx.token_seq, table, o_lat, H,
-                                         self.kv_rank, self.scale, window=self.window, gate=gate)
+                                         self.kv_rank, self.scale, window=self.window, gate=gate, sink=self.sink)
         else:
             splits = ctx.attention_splits(n * H)
             if self.window:  # a slice has at least 64 keys of the window
@@ -202,9 +218,10 @@ class LatentAttention(Part):
             partial = ws.get("attn_partial", (n * H * splits * (self.kv_rank + 2),), torch.float32) \
                 if splits > 1 else None
             ops.attention_latent(q_lat, cache.k, ctx.token_pos, ctx.token_seq, table, o_lat, H, self.kv_rank,
-                                 self.scale, splits, partial, window=self.window, gate=gate)
+                                 self.scale, splits, partial, window=self.window, gate=gate, sink=self.sink)
         attn = ws.get("attn", (n, H * self.vdim), self.dtype)
-        ops.batched_linear(o_lat, self.kv_rank, self.w_uv, attn, self.vdim)
+        ops.batched_linear(o_lat, self.kv_rank, self.w_uv, attn, self.vdim, gate=down if self.gate_by_value else None,
+                           gate_off=self.q_cols + self.row if self.gate_by_value else 0)
         linear(attn, self.w_o, None, residual, ADD_F32, ws, decode=ctx.decode)
 
     def _queries_from_latent(self, ctx, down, q_lat, freq, table, cache) -> None:

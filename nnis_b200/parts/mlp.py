@@ -9,7 +9,8 @@ params: hidden_size, intermediate_size, activation, bias, names {gate, up, down}
 Activations: "silu" (silu(gate) * up, fused into the products' epilogues where those
 exist) and "glu_clamp" with ``limit`` and ``alpha``: g' sigmoid(alpha g') (u' + 1) with
 g' = min(gate, limit), u' = up clamped to [-limit, limit] (in the tcgen05 product's epilogue where
-that product runs; a kernel of its own after a float32 product elsewhere).
+that product runs; a kernel of its own after a float32 product elsewhere); "gelu_tanh": gelu(gate) * up
+with gelu's tanh form, in the same places as silu.
 """
 from __future__ import annotations
 
@@ -31,8 +32,10 @@ class GatedMLP(Part):
         self.bias = bool(params.get("bias", False))
         self.names = params["names"]
         self.activation = params.get("activation", "silu")
-        if self.activation not in ("silu", "glu_clamp"):
+        if self.activation not in ("silu", "glu_clamp", "gelu_tanh"):
             raise ValueError(f"gated_mlp: activation {params['activation']!r} has no kernel")
+        # the decode kernels' code of the gate's activation (0: silu), where they have it
+        self.fused_act = {"silu": 0, "gelu_tanh": ops.GEMM_ACT_GELU_TANH}.get(self.activation)
         self.limit = float(params.get("limit", 0.0))
         self.alpha = float(params.get("alpha", 1.0))
         if self.activation == "glu_clamp" and not self.limit > 0:
@@ -69,7 +72,7 @@ class GatedMLP(Part):
 
     def _fused_gate_up(self, ctx, n: int, normed: bool = False) -> bool:
         """The fused bfloat16 decode kernel for gate/up (few rows, one token each)."""
-        return (self.dtype == torch.bfloat16 and ctx.decode and self.activation == "silu"
+        return (self.dtype == torch.bfloat16 and ctx.decode and self.fused_act is not None
                 and ops.gemv_pays(n, 2 * self.inter, self.hidden, ops.EPI_GATED, self.device, normed))
 
     def _fused_down(self, ctx, n: int) -> bool:
@@ -82,7 +85,7 @@ class GatedMLP(Part):
     def shares_norm(self, norm, ctx, n: int) -> bool:
         """Whether gate/up can end a norm that the projection before it began."""
         return (getattr(norm, "kind", None) == "rmsnorm" and self.dtype == torch.bfloat16 and ctx.decode
-                and self.activation == "silu"
+                and self.fused_act is not None
                 and ops.gemv_shares_norm(n, 2 * self.inter, self.hidden, ops.EPI_GATED, self.device))
 
     def forward(self, x: torch.Tensor, ctx, residual: torch.Tensor) -> None:
@@ -102,15 +105,18 @@ class GatedMLP(Part):
         act = ws.get("act", (n, self.inter), self.dtype)
         if begun is not None:
             ops.gemv_bf16(self.w_gu, self.b_gu, act, ops.EPI_GATED, x=begun.x, shares=begun.shares,
-                          eps=begun.norm.eps, m=n)
+                          eps=begun.norm.eps, m=n, act=self.fused_act)
         elif self._fused_gate_up(ctx, n, normed=hidden is not None):
             ops.gemv_bf16(self.w_gu, self.b_gu, act, ops.EPI_GATED, x=x, hidden=hidden,
                           norm_weight=norm.weight if norm is not None else None,
-                          eps=norm.eps if norm is not None else 0.0, m=n)
+                          eps=norm.eps if norm is not None else 0.0, m=n, act=self.fused_act)
         elif self.activation == "silu" and self.dtype == torch.bfloat16 \
                 and ops.gemm_tc_takes(n, 2 * self.inter, self.hidden):
             # tensor-core product with the activation in its epilogue
             ops.gemm_tc(x, self.w_gu, self.b_gu, act, ops.GEMM_GATED)
+        elif self.activation == "gelu_tanh" and self.dtype == torch.bfloat16 \
+                and ops.gemm_tc_takes(n, 2 * self.inter, self.hidden):
+            ops.gemm_tc_gelu_gated(x, self.w_gu, self.b_gu, act)
         elif self.activation == "glu_clamp" and self.dtype == torch.bfloat16 \
                 and ops.gemm_tc_takes(n, 2 * self.inter, self.hidden):
             # the same product with the clamped activation in its epilogue
@@ -120,6 +126,8 @@ class GatedMLP(Part):
             linear(x, self.w_gu, self.b_gu, gate_up, STORE_F32, decode=ctx.decode)
             if self.activation == "silu":
                 ops.silu_mul(gate_up, act)
+            elif self.activation == "gelu_tanh":
+                ops.gelu_mul(gate_up, act)
             else:
                 ops.glu_clamp(gate_up, act, self.limit, self.alpha)
         if self._fused_down(ctx, n):

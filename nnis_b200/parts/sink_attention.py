@@ -10,6 +10,7 @@ i reads key/value head i // (H / G)) with values of ``vdim``:
   head of q and of k is divided by its own root mean square AFTER the rotation, without a weight;
   with ``qk_norm == "head_weight"`` by its own root mean square BEFORE the rotation and multiplied by
   a weight per value of a head, which all heads share.
+* With ``values`` "keys" there is no W_v: the values are the keys as projected, before norm and rotation.
 * q and k are rotated by position (``dims`` 0: not at all) over the first ``dims`` values of every head (the
   position encoding's frequencies; neighbouring pairs, or, for an encoding whose ``pairing`` is
   "half", value i with value i + dims / 2).
@@ -41,7 +42,7 @@ key and value heads of 64 or of 128 run a tensor-core form of it (``attention_si
 
 params: hidden_size, heads, kv_heads, dim, vdim, scale, softcap, chunk, window, keep_first,
 distance_bias, sink, gate, qk_norm, head_scale, eps, position (a ``rope_frequencies`` PartSpec),
-pad_heads, kv ("own" | "shared"), names {q, k, v, o, q_norm, k_norm, sink, gate, head_scale, distance_bias}.
+pad_heads, values ("own" | "keys"), kv ("own" | "shared"), names {q, k, v, o, q_norm, k_norm, sink, gate, head_scale, distance_bias}.
 """
 from __future__ import annotations
 
@@ -118,6 +119,13 @@ class SinkAttention(Part):
         self.eps = float(params.get("eps", 1e-6))
         self.pad_heads = bool(params.get("pad_heads", False))
         self.own_kv = params.get("kv", "own") == "own"
+        values = params.get("values", "own")
+        if values not in ("own", "keys"):
+            raise ValueError(f"sink attention: values {values!r} is not known (own, keys)")
+        self.values_are_keys = values == "keys"
+        if self.values_are_keys and (self.dim != self.vdim or not self.own_kv or self.params.get("qk_norm") in (True, "whole")):
+            raise ValueError("sink attention: values that are the keys have their size, a cache of the layer's own and "
+                             "no norm over whole projections")
         self.names = params["names"]
         if self.heads % self.kv_heads:
             raise ValueError(f"heads={self.heads} is not a multiple of kv_heads={self.kv_heads}")
@@ -145,7 +153,9 @@ class SinkAttention(Part):
     def _projections(self):
         rows = [("q", self.heads * self.dim)]
         if self.own_kv:
-            rows += [("k", self.kv_heads * self.dim), ("v", self.kv_heads * self.vdim)]
+            rows.append(("k", self.kv_heads * self.dim))
+            if not self.values_are_keys:
+                rows.append(("v", self.kv_heads * self.vdim))
         if self.has_gate:
             rows.append(("gate", self.gate_cols))
         return rows
@@ -245,7 +255,9 @@ class SinkAttention(Part):
                      table if G else None, q, cache.k if G else None, cache.v if G else None, gate, H, G,
                      self.dim, self.vdim, self.position.dims, self.eps, pairing=self.pairing,
                      head_norm=self.head_norm, q_scale=self.head_scale,
-                     head_weights=None if whole else (self.q_norm, self.k_norm))
+                     magnitude=float(getattr(self.position, "magnitude", 1.0)),
+                     head_weights=None if whole else (self.q_norm, self.k_norm),
+                     values_are_keys=self.values_are_keys)
         out = ws.get("sink_attention_out", (n, H * self.vdim), self.dtype)
         if not ctx.decode and self._mma_prompt() and self.TILES_64 in ctx.tables:
             ops.attention_sink_mma(q, cache.k, cache.v, ctx.tables[self.TILES_64], ctx.seq_first_row, ctx.seq_start,
