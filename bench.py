@@ -3,7 +3,7 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--impl ours|reference]
                     [--shape 135m|360m|1.7b] [--batch B] [--context C] [--layers L] [--skip-points]
-                    [--skip-e2e] [--designs s,m [--only-design llama,nafezen,tazadra,sedopel,selovik,setenex]]
+                    [--skip-e2e] [--designs s,m [--only-design llama,nafezen,tazadra,sedopel,selovik,setenex,zadurax]]
 
 A step is one decode step of a batch of 8 sequences whose context ends at 4,096
 tokens (prompt 2,048 + 2,048 decoded); ``value`` is decoded tokens per second,
@@ -236,10 +236,10 @@ def timeline(engine, batch, path, rng, vocab):
 
 
 # ---------------------------------------------------------------------------
-# --designs: the Nafezen, Tazadra, Sedopel, Selovik and Setenex designs beside the Llama decoder at equal width and depth
+# --designs: the Nafezen, Tazadra, Sedopel, Selovik, Setenex and Zadurax designs beside the Llama decoder at equal width and depth
 # ---------------------------------------------------------------------------
 def design_configs(size: str):
-    """(Llama, Nafezen, Tazadra, Sedopel, Selovik, Setenex) configurations of one width, depth, vocabulary and dense
+    """(Llama, Nafezen, Tazadra, Sedopel, Selovik, Setenex, Zadurax) configurations of one width, depth, vocabulary and dense
     feed-forward size; the Nafezen layers alternate latent attention with dense and expert
     feed-forwards and hold one retention layer in four; the Tazadra layers are attention with a
     sink + dense, WKV + experts, selective scan + experts, and attention that reads the first
@@ -250,7 +250,9 @@ def design_configs(size: str):
     in turn, six layers of which the second and third run twice (eight layer runs); the Setenex layers
     alternate attention with a bias per distance (a window of 1,024 that keeps 64 first tokens) and latent
     attention with queries straight from the input and a window of 1,024, all with experts, six layers
-    of which the second and third run twice."""
+    of which the second and third run twice; the Zadurax layers are a matrix memory, latent attention with a
+    sink twice, and attention whose values are its keys (a window of 1,024), all with dense feed-forwards,
+    six layers of which the third and fourth run again with a cache of their own."""
     width, heads, ff, layers, q_rank, kv_rank, experts, top = {
         "s": (1024, 16, 2816, 8, 384, 256, 16, 2),
         "m": (2048, 16, 5632, 8, 768, 512, 32, 4),
@@ -321,10 +323,22 @@ def design_configs(size: str):
                  "mlp": x_moe} for i in range(layers - 2)]
     setenex = {"architecture": "Setenex", "vocab": 32768, "width": width, "norm": {"eps": 1e-5},
                "embedding": {"scale": 1.0}, "loop": {"start": 1, "stop": 3, "times": 2}, "layers": x_layers}
-    return llama, nafezen, tazadra, sedopel, selovik, setenex
+    memory = {"heads": ret_heads, "dim": 128, "vdim": 256, "gate_cap": 15.0}
+    sunk = {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "kv_rank": kv_rank,
+            "rot": {"base": 10000.0, "dims": dim // 2,
+                    "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}},
+            "scale": (dim + dim // 2) ** -0.5}
+    keyed = {"heads": heads, "kv_heads": heads // 4, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+             "mask": {"size": 1024}, "rot": {"base": 10000.0, "dims": dim // 2}}
+    pattern = [("mlstm", memory), ("latent_attention", sunk), ("latent_attention", sunk), ("attention", keyed)]
+    z_layers = [{"type": pattern[i % 4][0], "mixer": pattern[i % 4][1], "mlp": dense} for i in range(layers)]
+    for i in range(layers - 2, layers):
+        z_layers[i]["weights_of"] = i - 4
+    zadurax = {"architecture": "Zadurax", "vocab": 32768, "width": width, "norm": {"eps": 1e-6}, "layers": z_layers}
+    return llama, nafezen, tazadra, sedopel, selovik, setenex, zadurax
 
 
-DESIGN_NAMES = ("llama", "nafezen", "tazadra", "sedopel", "selovik", "setenex")
+DESIGN_NAMES = ("llama", "nafezen", "tazadra", "sedopel", "selovik", "setenex", "zadurax")
 
 
 def profile_steps(args) -> int:
@@ -511,10 +525,10 @@ def main() -> int:
     ap.add_argument("--shape", default="135m", choices=sorted(SHAPES),
                     help="layer sizes: the SmolLM2-135M shape (the benchmark) or a larger one of the family")
     ap.add_argument("--designs", metavar="SIZES", default=None,
-                    help="instead of the benchmark: the Nafezen, Tazadra, Sedopel, Selovik and Setenex designs beside the Llama decoder at "
+                    help="instead of the benchmark: the Nafezen, Tazadra, Sedopel, Selovik, Setenex and Zadurax designs beside the Llama decoder at "
                          "equal width and depth, sizes 's' and/or 'm' with commas: prefill, its parts, decoding")
     ap.add_argument("--only-design", metavar="NAMES", default=None,
-                    help="with --designs: only these of llama, nafezen, tazadra, sedopel, selovik, setenex (commas between them)")
+                    help="with --designs: only these of llama, nafezen, tazadra, sedopel, selovik, setenex, zadurax (commas between them)")
     ap.add_argument("--profile-steps", type=int, default=0,
                     help="with --designs: run this many eager prompt and decode steps of one design's first "
                          "four layers for a profiler instead of the timed comparison")

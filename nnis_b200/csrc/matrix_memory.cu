@@ -18,9 +18,9 @@
 //                  prefix maximum.  A warp per (chunk, head).
 //   memory_chunk   what a chunk adds by itself: U = sum_s exp(u_s - max u) k_s v_s^T, and the same of k
 //                  alone; all chunks side by side.
-//   memory_carry   the states between the chunks of a sequence, in order: with M = max(m, max u),
-//                  S <- exp(m - M) S + exp(max u - M) U, m <- b_end + M; the state before a chunk
-//                  replaces the chunk's own U, the last state goes to the slot.
+//   memory_chain   m between the chunks of a sequence, in order: with M = max(m, max u), m <- b_end + M.
+//   memory_carry   S and n between the chunks, in order: S <- exp(m - M) S + exp(max u - M) U; the state
+//                  before a chunk replaces the chunk's own U, the last state goes to the slot.
 //   memory_out     the outputs, all chunks side by side:
 //                  O_t = exp(m_before - M_t) S_before^T q_t + sum_{s <= t} exp(u_s - M_t) (q_t . k_s) v_s,
 //                  the denominator the same with n and without v.
@@ -300,15 +300,48 @@ memory_chunk_kernel(const float* __restrict__ a, int a_cols, const double* __res
     }
 }
 
-// A thread per element of S, then of n.
+// The running maximum from chunk to chunk of a sequence, in order (a warp per (sequence, head)): `before` of every chunk
+// but the first, the factors of the state before a chunk and of the chunk's own sum (`factors` float [n_chunks, H, 2]), and
+// the maximum that the step leaves.
+__global__ void __launch_bounds__(32)
+memory_chain_kernel(const double* __restrict__ ends, double* before, float* __restrict__ factors,
+                    float* __restrict__ max_state, const int* __restrict__ seq_slots, const int* __restrict__ seq_start,
+                    const int* __restrict__ seq_count, const int* __restrict__ seq_first_chunk, int H) {
+    const int seq = blockIdx.x, h = blockIdx.y, lane = threadIdx.x;
+    const int c0 = seq_first_chunk[seq], c1 = seq_first_chunk[seq + 1];
+    if (c1 <= c0) return;
+    double m = before[(size_t)c0 * H + h];
+    for (int c = c0; c < c1; c += 32) {  // 32 chunks at a time: a lane holds one chunk's gates
+        const bool in = c + lane < c1;
+        const size_t at = (size_t)min(c + lane, c1 - 1) * H + h;
+        const double b_end = ends[at * 2], u_max = ends[at * 2 + 1];
+        double mine = 0.0;
+        for (int j = 0; j < min(32, c1 - c); ++j) {
+            if (lane == j) mine = m;
+            m = fmax(m, __shfl_sync(0xffffffffu, u_max, j)) + __shfl_sync(0xffffffffu, b_end, j);
+        }
+        if (in) {
+            const double M = fmax(mine, u_max);
+            before[at] = mine;
+            factors[at * 2] = expf((float)(mine - M));
+            factors[at * 2 + 1] = expf((float)(u_max - M));
+        }
+    }
+    if (lane == 0)
+        max_state[((size_t)seq_slots[seq] * 2 + ((seq_start[seq] + seq_count[seq]) & 1)) * H + h] = (float)m;
+}
+
+// A thread per V elements of S, then of n (V = 4 where dim and dim * vdim are multiples of four).
+template <int V>
 __global__ void __launch_bounds__(256)
-memory_carry_kernel(float* chunk_state, float* chunk_norm, float* state, float* norm_state, float* max_state,
-                    const double* __restrict__ ends, double* before, const int* __restrict__ seq_slots,
+memory_carry_kernel(float* chunk_state, float* chunk_norm, float* state, float* norm_state,
+                    const float* __restrict__ factors, const int* __restrict__ seq_slots,
                     const int* __restrict__ seq_start, const int* __restrict__ seq_count,
                     const int* __restrict__ seq_first_chunk, int H, int dim, int vdim) {
     constexpr int AHEAD = 4;
+    struct alignas(4 * V) Pack { float x[V]; };
     const int seq = blockIdx.x, h = blockIdx.y, per = dim * vdim;
-    const int e = blockIdx.z * 256 + threadIdx.x;
+    const int e = (blockIdx.z * 256 + threadIdx.x) * V;
     if (e >= per + dim) return;
     const int c0 = seq_first_chunk[seq], c1 = seq_first_chunk[seq + 1];
     if (c1 <= c0) return;
@@ -319,26 +352,22 @@ memory_carry_kernel(float* chunk_state, float* chunk_norm, float* state, float* 
     float* from = is_n ? norm_state + ((size_t)slot * 2 + (start & 1)) * H * dim + (size_t)h * dim + (e - per)
                        : state + ((size_t)slot * H + h) * per + e;
     float* to = is_n ? norm_state + ((size_t)slot * 2 + (end & 1)) * H * dim + (size_t)h * dim + (e - per) : from;
-    double m = before[(size_t)c0 * H + h];
-    float run = *from;
+    Pack run = *reinterpret_cast<const Pack*>(from);
     for (int c = c0; c < c1; c += AHEAD) {
-        float add[AHEAD];
+        Pack add[AHEAD];
 #pragma unroll
         for (int j = 0; j < AHEAD; ++j)
-            if (c + j < c1) add[j] = own[(size_t)(c - c0 + j) * step];
+            if (c + j < c1) add[j] = *reinterpret_cast<const Pack*>(own + (size_t)(c - c0 + j) * step);
 #pragma unroll
         for (int j = 0; j < AHEAD; ++j) {
             if (c + j >= c1) break;
-            const double b_end = ends[((size_t)(c + j) * H + h) * 2], u_max = ends[((size_t)(c + j) * H + h) * 2 + 1];
-            if (e == 0 && c + j > c0) before[(size_t)(c + j) * H + h] = m;
-            const double M = fmax(m, u_max);
-            own[(size_t)(c - c0 + j) * step] = run;
-            run = fmaf(expf((float)(m - M)), run, expf((float)(u_max - M)) * add[j]);
-            m = b_end + M;
+            const float2 f = *reinterpret_cast<const float2*>(factors + ((size_t)(c + j) * H + h) * 2);
+            *reinterpret_cast<Pack*>(own + (size_t)(c - c0 + j) * step) = run;
+#pragma unroll
+            for (int v = 0; v < V; ++v) run.x[v] = fmaf(f.x, run.x[v], f.y * add[j].x[v]);
         }
     }
-    *to = run;
-    if (e == 0) max_state[((size_t)slot * 2 + (end & 1)) * H + h] = (float)m;
+    *reinterpret_cast<Pack*>(to) = run;
 }
 
 // A CTA of 256 threads per (chunk, head, BV columns of vdim).  Scores: 4 x 4 a thread; outputs: 4 columns and
@@ -541,9 +570,18 @@ static cudaError_t launch_memory_prompt(const float* a, int a_cols, float* state
     const int v_tiles = (vdim + BV - 1) / BV, d_tiles = (dim + 63) / 64;
     memory_chunk_kernel<BV><<<dim3(n_chunks, H, v_tiles * d_tiles), 256, 0, stream>>>(
         a, a_cols, u, ends, chunks, seq_first_row, seq_count, chunk_state, chunk_norm, H, dim, vdim);
-    memory_carry_kernel<<<dim3(n_seqs, H, (dim * vdim + dim + 255) / 256), 256, 0, stream>>>(
-        chunk_state, chunk_norm, state, norm_state, max_state, ends, before, seq_slots, seq_start, seq_count,
-        seq_first_chunk, H, dim, vdim);
+    float* factors = reinterpret_cast<float*>(chunk_gates + (size_t)3 * n_chunks * H);
+    memory_chain_kernel<<<dim3(n_seqs, H), 32, 0, stream>>>(ends, before, factors, max_state, seq_slots, seq_start,
+                                                            seq_count, seq_first_chunk, H);
+    const int elems = dim * vdim + dim;
+    if (dim % 4 == 0)
+        memory_carry_kernel<4><<<dim3(n_seqs, H, (elems / 4 + 255) / 256), 256, 0, stream>>>(
+            chunk_state, chunk_norm, state, norm_state, factors, seq_slots, seq_start, seq_count, seq_first_chunk, H, dim,
+            vdim);
+    else
+        memory_carry_kernel<1><<<dim3(n_seqs, H, (elems + 255) / 256), 256, 0, stream>>>(
+            chunk_state, chunk_norm, state, norm_state, factors, seq_slots, seq_start, seq_count, seq_first_chunk, H, dim,
+            vdim);
     const size_t smem = (size_t)(2 * 32 * (kMemChunk + 4) + kMemChunk * (kMemChunk + 4) + 32 * BV) * sizeof(float);
     auto kernel = memory_out_kernel<BV>;
     if (smem > 48 * 1024) {
@@ -587,7 +625,7 @@ NNIS_API int nnis_memory_step(const float* a, int a_cols, const float* i_bias, c
 
 // Prompt steps.  chunks: int32 [n_chunks, 2] = (sequence, first token of the chunk among the sequence's tokens of this
 // step), 64 tokens each but for a sequence's last, in the order of the sequences; seq_first_chunk
-// [n_seqs + 1].  Scratch: gates double [3, n_tokens, H]; chunk_gates double [3, n_chunks, H]; chunk_state
+// [n_seqs + 1].  Scratch: gates double [3, n_tokens, H]; chunk_gates double [4, n_chunks, H]; chunk_state
 // float32 [n_chunks, H, dim, vdim]; chunk_norm float32 [n_chunks, H, dim].
 NNIS_API int nnis_memory_prompt(const float* a, int a_cols, const float* i_bias, const float* f_bias, float* state,
                                 float* norm_state, float* max_state, const int* chunks, int n_chunks,

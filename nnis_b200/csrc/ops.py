@@ -2151,7 +2151,7 @@ def memory_prompt(a: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, s
                   chunk_state: torch.Tensor, chunk_norm: torch.Tensor, o_raw: torch.Tensor, heads: int, dim: int,
                   vdim: int, cap: float, q_scale: float, floor: float) -> None:
     """``memory_step`` for prompt steps, chunk by chunk (``scan_segments`` of ``memory_chunk_tokens``).  Scratch:
-    ``gates`` float64 [3, n, heads], ``chunk_gates`` float64 [3, chunks, heads], ``chunk_state`` float32
+    ``gates`` float64 [3, n, heads], ``chunk_gates`` float64 [4, chunks, heads], ``chunk_state`` float32
     [chunks, heads, dim, vdim], ``chunk_norm`` float32 [chunks, heads, dim]."""
     _cuda(a, i_bias, f_bias, state, norm_state, max_state, chunks, seq_first_chunk, seq_slots, seq_first_row, seq_start,
           seq_count, gates, chunk_gates, chunk_state, chunk_norm, o_raw)
@@ -2160,7 +2160,7 @@ def memory_prompt(a: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, s
     _need(chunks.dtype == torch.int32 and chunks.dim() == 2 and chunks.shape[1] == 2
           and seq_first_chunk.dtype == torch.int32 and seq_first_chunk.numel() == seqs + 1, "memory_prompt: chunk lists")
     _need(gates.dtype == chunk_gates.dtype == torch.float64 and gates.numel() >= 3 * n * heads
-          and chunk_gates.numel() >= 3 * c * heads, "memory_prompt: float64 gate scratch")
+          and chunk_gates.numel() >= 4 * c * heads, "memory_prompt: float64 gate scratch")
     _need(chunk_state.dtype == chunk_norm.dtype == torch.float32 and chunk_state.numel() >= c * heads * dim * vdim
           and chunk_norm.numel() >= c * heads * dim, "memory_prompt: chunk scratch")
     _check(_lib().nnis_memory_prompt(_ptr(a), a.shape[1], _ptr(i_bias), _ptr(f_bias), _ptr(state), _ptr(norm_state),
@@ -2168,7 +2168,7 @@ def memory_prompt(a: torch.Tensor, i_bias: torch.Tensor, f_bias: torch.Tensor, s
                                      _ptr(seq_first_row), _ptr(seq_start), _ptr(seq_count), _ptr(gates),
                                      _ptr(chunk_gates), _ptr(chunk_state), _ptr(chunk_norm), _ptr(o_raw), n, heads, dim,
                                      vdim, ctypes.c_float(cap), ctypes.c_float(q_scale), ctypes.c_float(floor),
-                                     _stream()), "memory_prompt", 4)
+                                     _stream()), "memory_prompt", 5)
 
 
 def memory_finish(o_raw: torch.Tensor, a: torch.Tensor, gate_off: int, weight: torch.Tensor, token_pos: torch.Tensor,

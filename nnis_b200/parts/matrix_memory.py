@@ -123,7 +123,7 @@ class MatrixMemory(Part):
             ops.memory_prompt(rows, self.i_bias, self.f_bias, cache.state, norm_state, max_state, chunks,
                               ctx.tables[self.FIRST_CHUNK], ctx.seq_slots, ctx.seq_first_row, ctx.seq_start,
                               ctx.seq_count, ws.get("memory_gates", (3, n, H), torch.float64),
-                              ws.get("memory_chunk_gates", (3, c, H), torch.float64),
+                              ws.get("memory_chunk_gates", (4, c, H), torch.float64),
                               ws.get("memory_chunk_state", (c, H, self.dim, self.vdim), torch.float32),
                               ws.get("memory_chunk_norm", (c, H, self.dim), torch.float32), o_raw, *sizes)
         gated = ws.get("memory_gated", (n, H * self.vdim), self.dtype)
