@@ -338,7 +338,7 @@ memory_carry_kernel(float* chunk_state, float* chunk_norm, float* state, float* 
                     const float* __restrict__ factors, const int* __restrict__ seq_slots,
                     const int* __restrict__ seq_start, const int* __restrict__ seq_count,
                     const int* __restrict__ seq_first_chunk, int H, int dim, int vdim) {
-    constexpr int AHEAD = 4;
+    constexpr int AHEAD = 8;
     struct alignas(4 * V) Pack { float x[V]; };
     const int seq = blockIdx.x, h = blockIdx.y, per = dim * vdim;
     const int e = (blockIdx.z * 256 + threadIdx.x) * V;
@@ -373,7 +373,7 @@ memory_carry_kernel(float* chunk_state, float* chunk_norm, float* state, float* 
 // A CTA of 256 threads per (chunk, head, BV columns of vdim).  Scores: 4 x 4 a thread; outputs: 4 columns and
 // BV / 16 rows a thread.
 template <int BV>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 memory_out_kernel(const float* __restrict__ a, int a_cols, const double* __restrict__ b, const double* __restrict__ u,
                   const double* __restrict__ top, const double* __restrict__ before,
                   const float* __restrict__ chunk_state, const float* __restrict__ chunk_norm,
@@ -588,6 +588,9 @@ static cudaError_t launch_memory_prompt(const float* a, int a_cols, float* state
         cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return e;
     }
+    cudaError_t carve = cudaFuncSetAttribute(kernel, cudaFuncAttributePreferredSharedMemoryCarveout,
+                                             cudaSharedmemCarveoutMaxShared);  // three CTAs an SM
+    if (carve != cudaSuccess) return carve;
     kernel<<<dim3(n_chunks, H, v_tiles), 256, smem, stream>>>(a, a_cols, b, u, top, before, chunk_state, chunk_norm,
                                                               chunks, seq_first_row, seq_start, seq_count, o_raw, H,
                                                               dim, vdim, q_scale, floor_add);
